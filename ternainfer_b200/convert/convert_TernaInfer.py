@@ -21,6 +21,7 @@ Hugging-Face download/renaming half of the reference script is not rebuilt.
 from __future__ import annotations
 
 import argparse
+import json
 import os
 from typing import Dict
 
@@ -150,6 +151,15 @@ def random_checkpoint(dim: int, n_layers: int, n_heads: int, n_kv_heads: int, ff
     return dic
 
 
+def write_config(folder: str, state: Dict[str, torch.Tensor], dim: int, n_heads: int, n_kv_heads: int, ffn_dim: int):
+    """``config.json`` beside the weights, as ``registry.load_model`` reads it."""
+    layers = {int(k.split(".")[1]) for k in state if k.startswith("layers.")}
+    cfg = {"architecture": "TernaInfer", "dim": dim, "n_layers": len(layers), "n_heads": n_heads, "n_kv_heads": n_kv_heads,
+           "ffn_dim": ffn_dim, "vocab_size": state["tok_embeddings.weight"].shape[0], "fused_glue": True}
+    with open(os.path.join(folder, "config.json"), "w") as f:
+        json.dump(cfg, f, indent=1)
+
+
 def main():
     ap = argparse.ArgumentParser(description="fused-name state dict (.pt or .safetensors) -> TernaInfer checkpoint files")
     ap.add_argument("--input", required=True)
@@ -172,6 +182,7 @@ def main():
     ternary, other = pack_state_dict(int8_state, a.device)
     torch.save(ternary, os.path.join(a.output_dir, "model_TernaInfer_TernaryWeights.pt"))
     torch.save(other, os.path.join(a.output_dir, "model_embeddings_and_norms_non_ternary.pt"))
+    write_config(a.output_dir, state, a.dim, a.n_heads, a.n_kv_heads, a.ffn_dim)
     print(f"saved {len(ternary) // 4} packed weights to {a.output_dir}")
 
 

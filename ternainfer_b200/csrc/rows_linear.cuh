@@ -1,0 +1,78 @@
+// Dense bf16 linear for decode-sized batches (up to 8 rows) on sm_100a: out[m][n] = act(sum_k W[n][k] x[m][k]).
+//
+// HBM-bound: W is read exactly once.  A CTA owns 16 rows of W; its eight warps split K, each streaming its
+// slice with one 128-bit load per lane and row (lane (g, q) of the MMA holds rows g and g+8, 8 consecutive k
+// starting at 8q; k is only a summation index, so the fragments of mma.sync m16n8k16 are filled straight from
+// those registers, as in lm_head.cuh).  The first kRowsPre k-steps of W are requested before the wait for the
+// previous kernel of the stream, so the weights' latency runs underneath its tail.  The rows of x are the
+// MMA's N = 8 and come from L2.  Warp partials meet in shared memory in a fixed order.
+#pragma once
+#include "decoder_common.cuh"
+#include "lm_head.cuh"
+
+namespace tsp {
+
+constexpr int kRowsWarps = 8;
+constexpr int kRowsPre = 8;   // k-steps of 32 whose weights are in flight per warp
+
+struct RowsLinearParams {
+    const bf16* x;     // [M][K]
+    const bf16* w;     // [N][K]
+    void* out;         // [M][N] bf16 or fp32
+    int M, N, K;       // M <= 8, K a multiple of 8
+    int act;           // 1: square of relu
+};
+
+template <typename O>
+__global__ void __launch_bounds__(kRowsWarps * 32) rows_linear_kernel(const RowsLinearParams p) {
+    __shared__ float part[kRowsWarps][16][9];
+    griddep_launch_dependents();
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int g = lane >> 2, q = lane & 3;
+    const int K = p.K, steps = (K + 31) >> 5;
+    const int n0 = blockIdx.x * 16;
+    const int s0 = steps * warp / kRowsWarps, s1 = steps * (warp + 1) / kRowsWarps;
+    const bool ok0 = n0 + g < p.N, ok1 = n0 + g + 8 < p.N;
+    const bf16* w0 = p.w + (size_t)(ok0 ? n0 + g : 0) * K + q * 8;
+    const bf16* w1 = p.w + (size_t)(ok1 ? n0 + g + 8 : 0) * K + q * 8;
+    const bf16* x = p.x + (size_t)(g < p.M ? g : 0) * K + q * 8;
+    const bool xok = g < p.M;
+    const uint4 zero = make_uint4(0, 0, 0, 0);
+    uint4 a[kRowsPre], b[kRowsPre];
+    auto fetch = [&](int u, int s) {
+        const bool in = s < s1 && 32 * s + q * 8 < K;
+        a[u] = in ? ldg_stream_128(w0 + 32 * s) : zero;
+        b[u] = in ? ldg_stream_128(w1 + 32 * s) : zero;
+    };
+#pragma unroll
+    for (int u = 0; u < kRowsPre; ++u) fetch(u, s0 + u);
+    griddep_wait();
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+    for (int s = s0; s < s1; s += kRowsPre) {
+        uint4 xv[kRowsPre];
+#pragma unroll
+        for (int u = 0; u < kRowsPre; ++u)
+            xv[u] = (xok && s + u < s1 && 32 * (s + u) + q * 8 < K) ? ld_cg_128(x + 32 * (s + u)) : zero;
+#pragma unroll
+        for (int u = 0; u < kRowsPre; ++u) {
+            mma_bf16_16x8x16(acc, a[u].x, b[u].x, a[u].y, b[u].y, xv[u].x, xv[u].y);
+            mma_bf16_16x8x16(acc, a[u].z, b[u].z, a[u].w, b[u].w, xv[u].z, xv[u].w);
+            fetch(u, s + kRowsPre + u);
+        }
+    }
+    part[warp][g][2 * q] = acc[0], part[warp][g][2 * q + 1] = acc[1];
+    part[warp][g + 8][2 * q] = acc[2], part[warp][g + 8][2 * q + 1] = acc[3];
+    __syncthreads();
+    if (tid < 128) {
+        const int r = tid & 15, t = tid >> 4;
+        if (t < p.M && n0 + r < p.N) {
+            float v = 0.f;
+#pragma unroll
+            for (int i = 0; i < kRowsWarps; ++i) v += part[i][r][t];
+            if (p.act == 1) v = fmaxf(v, 0.f), v *= v;
+            reinterpret_cast<O*>(p.out)[(size_t)t * p.N + n0 + r] = from_f<O>(v);
+        }
+    }
+}
+
+}  // namespace tsp

@@ -1,20 +1,25 @@
-"""ctypes binding of ``libternaspmm.so`` (built in-tree under ``csrc/``).
+"""ctypes bindings of ``libternaspmm.so`` and ``libdecoderops.so`` (built in-tree under ``csrc/``).
 
 The reference binds its library with ``ctypes.CDLL('./kernels/libternaspmm.so')``
 and passes every pointer as ``c_void_p`` (model.py:21, :76-89 of
 Gu-J/TernaInfer); this module does the same against the B200 library and
 declares argument types so that mistakes fail in Python rather than on the GPU.
 There is no fallback: if the library is missing, loading raises.
+``libdecoderops.so`` (include/decoder_ops.h) holds the kernels of the dense
+decoders; its calls take argument structs and return a status, which
+``check`` turns into an exception.
 """
 from __future__ import annotations
 
 import ctypes
+import fcntl
 import os
 import subprocess
 
 _HERE = os.path.dirname(os.path.abspath(__file__))
 _CSRC = os.path.join(_HERE, "csrc")
 _LIB = None
+_DECODER_LIB = None
 
 _P = ctypes.c_void_p
 _I = ctypes.c_int
@@ -28,14 +33,82 @@ class ListItem(ctypes.Structure):
                [(n, _I) for n in ("ws_num", "M", "N", "K", "seg1", "seg2", "seg3", "prefill_form")]
 
 
+def _struct(name, fields):
+    """``fields``: 'type: names' lines in the order of the C struct."""
+    kinds = {"p": _P, "i": _I, "l": ctypes.c_longlong, "f": ctypes.c_float}
+    flat = [(n, kinds[line[0]]) for line in fields for n in line[2:].split()]
+    return type(name, (ctypes.Structure,), {"_fields_": flat})
+
+
+# the argument structs of include/decoder_ops.h
+EmbedArgs = _struct("EmbedArgs", ["p tokens pos prev embed bigram x", "l mul_prev mul_cur buckets", "i B T S D V"])
+HyperArgs = _struct("HyperArgs", ["p x y mix out in_ w rows h", "f m w_offset eps", "i D S n_rows"])
+DeltaArgs = _struct("DeltaArgs", ["p proj zw w2 w0 a_bias norm pos state o y", "i B T H dk dv rank", "l ld",
+                                  "i off_r off_k off_v off_a off_g off_w1", "f eps"])
+AttnArgs = _struct("AttnArgs", ["p proj ck cv q_norm k_norm bias slope pos y", "i B T H G dim vdim", "l ld",
+                                "i off_q off_k off_v off_g", "i chunk slots", "f scale eps"])
+
+
 def library_path() -> str:
     return os.path.join(_CSRC, "libternaspmm.so")
 
 
+def decoder_library_path() -> str:
+    return os.path.join(_CSRC, "libdecoderops.so")
+
+
 def build_library(verbose: bool = False) -> str:
-    """Compile the library for sm_100a with nvcc (``make -C csrc``)."""
+    """Compile the libraries for sm_100a with nvcc (``make -C csrc``)."""
     subprocess.run(["make", "-C", _CSRC] + (["verbose"] if verbose else []), check=True)
     return library_path()
+
+
+def build_decoder_library() -> str:
+    """Compile ``libdecoderops.so`` alone, if it is not up to date; safe to call from several processes."""
+    with open(os.path.join(_CSRC, "Makefile")) as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        subprocess.run(["make", "-C", _CSRC, "libdecoderops.so"], check=True, stdout=subprocess.DEVNULL)
+    return decoder_library_path()
+
+
+class DecoderOpsError(RuntimeError):
+    """A call into ``libdecoderops.so`` was refused; the library has written the reason to stderr."""
+
+
+def check(status: int):
+    if status:
+        raise DecoderOpsError({1: "shape not supported", 2: "bad pointer", 3: "launch failed"}.get(status, str(status)))
+
+
+def load_decoder_library() -> ctypes.CDLL:
+    """Load ``libdecoderops.so``; raises ``OSError`` if it has not been built."""
+    global _DECODER_LIB
+    if _DECODER_LIB is not None:
+        return _DECODER_LIB
+    path = decoder_library_path()
+    if not os.path.exists(path):
+        raise OSError(f"{path} not found: build it with `make -C {_CSRC} libdecoderops.so` (or __graft_entry__.build())")
+    lib = ctypes.CDLL(path)
+    L = ctypes.c_longlong
+    for name, args in (("decoder_embed", [ctypes.POINTER(EmbedArgs), _I, _I, _P]),
+                       ("decoder_hyper", [ctypes.POINTER(HyperArgs), _I, _I, _P]),
+                       ("decoder_rows_linear", [_P, _P, _P, _I, _I, _I, _I, _I, _I, _P]),
+                       ("decoder_head_argmax", [_P, _P, _I, _I, _I, _P, _P, _P, _P]),
+                       ("decoder_relu2", [_P, L, _I, _I, _P]),
+                       ("decoder_delta", [ctypes.POINTER(DeltaArgs), _I, _I, _P]),
+                       ("decoder_tanh_cols", [_P, L, _I, _I, L, _P, _I, _I, _P]),
+                       ("decoder_attn", [ctypes.POINTER(AttnArgs), _I, _I, _I, _P])):
+        fn = getattr(lib, name)
+        fn.argtypes = args
+        fn.restype = _I
+    lib.decoder_head_scratch_bytes.argtypes = []
+    lib.decoder_head_scratch_bytes.restype = L
+    _DECODER_LIB = lib
+    return lib
+
+
+DECODER_SYMBOLS = ("decoder_embed", "decoder_hyper", "decoder_rows_linear", "decoder_head_scratch_bytes",
+                   "decoder_head_argmax", "decoder_relu2", "decoder_delta", "decoder_tanh_cols", "decoder_attn")
 
 
 def load_library() -> ctypes.CDLL:

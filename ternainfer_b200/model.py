@@ -20,6 +20,7 @@ import torch
 from torch import nn
 from torch.nn import functional as F
 
+from .cache import SequenceCache
 from .linear import SpBitLinear, quant_input, rmsnorm, rmsnorm_quant, lm_head_argmax
 
 
@@ -233,13 +234,17 @@ class Transformer(nn.Module):
                     raise
                 self.flash = False
 
-    def make_cache(self, batch: int, device, dtype=torch.bfloat16) -> List[LayerCache]:
+    @property
+    def vocab_size(self) -> int:
+        return self.args.vocab_size
+
+    def make_cache(self, batch: int, device, dtype=torch.bfloat16) -> SequenceCache:
         a = self.args
         shape = (batch, a.n_kv_heads // self.tp, self.max_seq_len, a.head_dim)
         if self.flash:
             shape = (batch, self.max_seq_len, a.n_kv_heads, a.head_dim)
-        return [(torch.zeros(shape, device=device, dtype=dtype), torch.zeros(shape, device=device, dtype=dtype))
-                for _ in range(a.n_layers)]
+        return SequenceCache([(torch.zeros(shape, device=device, dtype=dtype),
+                               torch.zeros(shape, device=device, dtype=dtype)) for _ in range(a.n_layers)])
 
     def head(self, h: torch.Tensor, greedy: bool = False):
         """Final norm + tied output head.  fp32 logits [B, T, vocab] (model.py:380-386 of the
@@ -258,10 +263,11 @@ class Transformer(nn.Module):
         logits = F.linear(h, emb).float()
         return (None, logits.argmax(-1)) if greedy else logits
 
-    def forward(self, tokens: torch.Tensor, cache: List[LayerCache], pos: torch.Tensor, greedy_last: bool = False):
+    def forward(self, tokens: torch.Tensor, cache: List[LayerCache], pos: torch.Tensor, greedy_last: bool = False,
+                want: Optional[torch.Tensor] = None):
         """tokens [B, T]; pos [T] (device int64) = positions written in the cache.
-        Returns fp32 logits [B, T, vocab] (model.py:380-386 of the reference); with ``greedy_last``
-        only the greedy token of every sequence's last position, int64 [B] (what the generation
+        Returns fp32 logits [B, T, vocab] (model.py:380-386 of the reference), or [B, len(want), vocab]
+        at the places ``want`` (device int64) among the T; with ``greedy_last`` only the greedy token of every sequence's last position, int64 [B] (what the generation
         loop needs: generate.py:274, :283, :305 of the reference)."""
         if self._rope is None or self._rope[0].device != tokens.device:
             self._rope = rope_tables(self.args.head_dim, self.max_seq_len, self.args.rope_theta, tokens.device)
@@ -280,4 +286,4 @@ class Transformer(nn.Module):
             h = layer(h, c, pos, cos, sin, mask, fused, flash)
         if greedy_last:
             return self.head(h[:, -1:], greedy=True)[1][:, 0]
-        return self.head(h)
+        return self.head(h if want is None else h.index_select(1, want))
