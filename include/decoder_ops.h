@@ -5,7 +5,7 @@
  * Conventions.  All pointers are device pointers unless said otherwise.  dtype: the activation (and table)
  * type, 0 = bf16, 1 = fp32; parameters that enter 32-bit arithmetic (norm weights, biases, mixing weights)
  * are fp32.  Every call returns 0 or one of the codes below and launches nothing when it fails; nothing is
- * allocated and nothing synchronises, so all of it can be captured in a CUDA graph.  pdl != 0: launch with
+ * allocated and nothing but decoder_status synchronises, so all of it can be captured in a CUDA graph.  pdl != 0: launch with
  * programmatic dependent launch (decode steps: the kernels' weight fetches start under their predecessor).
  * Positions are read from device memory (pos[0] = position of the call's first token in its sequence; all
  * sequences of a call are at the same position); position 0 starts a sequence: recurrent state and token
@@ -21,6 +21,11 @@ extern "C" {
 #define DECODER_BAD_SHAPE 1
 #define DECODER_BAD_POINTER 2
 #define DECODER_LAUNCH 3
+#define DECODER_WAIT_TIMEOUT 4
+
+/* Device-side status since the last call (synchronises): 0, or DECODER_WAIT_TIMEOUT when a bounded wait inside a
+ * kernel ran out, in which case that kernel's output is incomplete. */
+int decoder_status(void);
 
 /* x[row][s][:] = embed[token] + bigram[(previous * mul_prev + token * mul_cur) mod buckets], the same for all
  * S streams; a sequence's first token takes bigram row number `buckets`.  prev [B]: token before this call's

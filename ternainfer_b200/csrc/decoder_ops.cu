@@ -10,6 +10,7 @@
 #include "hyper.cuh"
 #include "rows_linear.cuh"
 #include "sigmoid_attn.cuh"
+#include "sigmoid_attn_tc.cuh"
 
 namespace tsp {
 
@@ -131,12 +132,47 @@ static int attn_one_l(const AttnParams& p, int pdl, void* stream) {
     return DECODER_BAD_SHAPE;
 }
 
+static bool encode_rows(CUtensorMap* map, const void* base, long long rows, long long cols, long long ld) {
+    typedef CUresult (*EncodeFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
+                                 const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
+                                 CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+    static EncodeFn fn = nullptr;
+    if (!fn) {
+        void* ptr = nullptr;
+        cudaDriverEntryPointQueryResult q;
+        if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &ptr, cudaEnableDefault, &q) != cudaSuccess || !ptr) return false;
+        fn = reinterpret_cast<EncodeFn>(ptr);
+    }
+    const cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows}, strides[1] = {(cuuint64_t)ld * 2};
+    const cuuint32_t box[2] = {64, 128}, step[2] = {1, 1};
+    return fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, step, CU_TENSOR_MAP_INTERLEAVE_NONE,
+              CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
+}
+
+// 16-byte starts for every tile, whole MMA steps: what the tensor-core kernel asks of a call
+static bool attn_tc_fits(const AttnParams& p) {
+    return p.dim % 16 == 0 && p.vdim % 16 == 0 && p.dim <= 128 && p.vdim <= 128 && p.ld % 8 == 0 && p.off_q % 8 == 0 && p.off_k % 8 == 0 &&
+           p.off_v % 8 == 0 && p.off_g % 8 == 0 && !misaligned(p.proj, 16) && !misaligned(p.ck, 16) && !misaligned(p.cv, 16) &&
+           !misaligned(p.y, 16);
+}
+
+static int attn_tc(const AttnParams& p, void* stream) {
+    CUtensorMap proj, ck, cv;
+    const long long cache_rows = (long long)p.B * p.G * p.slots;
+    if (!encode_rows(&proj, p.proj, (long long)p.B * p.T, p.ld, p.ld) || !encode_rows(&ck, p.ck, cache_rows, p.dim, p.dim) ||
+        !encode_rows(&cv, p.cv, cache_rows, p.vdim, p.vdim))
+        return bad(DECODER_LAUNCH, "attn: tensor map refused");
+    const int smem = AttnTcSmem::total((p.dim + 63) / 64, (p.vdim + 63) / 64);
+    return launch(sigmoid_attn_tc_kernel, dim3((p.T + 127) / 128, p.H, p.B), AttnTcSmem::threads, (size_t)smem, 0, stream, 1, p, proj, ck, cv);
+}
+
 template <typename A>
-static int attn_prompt(const AttnParams& p, int pdl, void* stream) {
+static int attn_prompt(const AttnParams& p, bool tensor_cores, int pdl, void* stream) {
     const long long units = (long long)p.B * p.T * (p.H + p.G);
     int rc = launch(head_norm_kernel<A>, dim3((unsigned)((units + 7) / 8)), 256, 0, pdl, stream, 1, p);
     if (rc) return rc;
-    rc = launch(sigmoid_attn_plain_kernel<A>, dim3(p.T, p.H, p.B), 128, (size_t)(p.dim + p.vdim) * 4, pdl, stream, 1, p);
+    rc = tensor_cores ? attn_tc(p, stream)
+                      : launch(sigmoid_attn_plain_kernel<A>, dim3(p.T, p.H, p.B), 128, (size_t)(p.dim + p.vdim) * 4, pdl, stream, 1, p);
     if (rc) return rc;
     return launch(attn_cache_store_kernel<A>, dim3(std::min(p.T, p.slots), p.B), 128, 0, pdl, stream, 1, p);
 }
@@ -230,5 +266,15 @@ extern "C" int decoder_attn(const decoder_attn_args* a, int dtype, int path, int
         if (widest <= 128) return attn_one_l<16>(*a, pdl, stream);
         return attn_one_l<32>(*a, pdl, stream);
     }
-    return dtype ? attn_prompt<float>(*a, pdl, stream) : attn_prompt<bf16>(*a, pdl, stream);
+    return dtype ? attn_prompt<float>(*a, false, pdl, stream) : attn_prompt<bf16>(*a, path == 0 && attn_tc_fits(*a), pdl, stream);
+}
+
+extern "C" int decoder_status(void) {
+    int v = 0;
+    if (cudaMemcpyFromSymbol(&v, g_decoder_status, sizeof(v)) != cudaSuccess) return DECODER_LAUNCH;
+    if (v) {
+        const int zero = 0;
+        cudaMemcpyToSymbol(g_decoder_status, &zero, sizeof(zero));
+    }
+    return v;
 }

@@ -42,9 +42,8 @@
 // its own accumulators and runs the epilogue for its columns.  (Remote
 // atomics were measured at 1-2 per clock per SM and are not used here.)
 #pragma once
-#include <cuda.h>
-
 #include "spmm_small_m.cuh"
+#include "tcgen05_sm100.cuh"
 
 namespace tsp {
 
@@ -73,79 +72,6 @@ struct LargeMSmem {
     static constexpr int align = DENSE ? 1024 : kLutBytes;          // the stage buffers need 1024 bytes, the tables 32 KB
     static constexpr int total = tables * kLutBytes + align + rest;   // tables first (aligned), the rest behind them
 };
-
-// ---- tcgen05 wrappers ------------------------------------------------------
-__device__ __forceinline__ void tc_fence_before() { asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory"); }
-__device__ __forceinline__ void tc_fence_after() { asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory"); }
-__device__ __forceinline__ void fence_proxy_async_smem() { asm volatile("fence.proxy.async.shared::cta;" ::: "memory"); }
-
-__device__ __forceinline__ void tmem_alloc(uint32_t slot_smem, uint32_t cols) {
-    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(slot_smem), "r"(cols)
-                 : "memory");
-    asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
-}
-__device__ __forceinline__ void tmem_dealloc(uint32_t taddr, uint32_t cols) {
-    asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(taddr), "r"(cols) : "memory");
-}
-// D[tmem] (+)= A[smem] * B[smem]; int8 operands, int32 accumulators, M=128, N and K=32 from the descriptors
-__device__ __forceinline__ void umma_i8(uint32_t d_tmem, uint64_t adesc, uint64_t bdesc, uint32_t idesc,
-                                        uint32_t accumulate) {
-    asm volatile(
-        "{ .reg .pred p; setp.ne.b32 p, %4, 0;\n"
-        "tcgen05.mma.cta_group::1.kind::i8 [%0], %1, %2, %3, p; }" ::"r"(d_tmem),
-        "l"(adesc), "l"(bdesc), "r"(idesc), "r"(accumulate)
-        : "memory");
-}
-__device__ __forceinline__ void umma_commit(uint32_t bar) {
-    asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(bar) : "memory");
-}
-__device__ __forceinline__ void tmem_ld16(uint32_t taddr, int (&v)[16]) {
-    asm volatile(
-        "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
-        : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]), "=r"(v[8]),
-          "=r"(v[9]), "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15])
-        : "r"(taddr));
-    asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-}
-// 2-D TMA tile load, completion in bytes on an mbarrier (no multicast)
-__device__ __forceinline__ void tma_load_2d(uint32_t dst, const CUtensorMap* map, int c0, int c1, uint32_t bar) {
-    asm volatile(
-        "cp.async.bulk.tensor.2d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];" ::
-            "r"(dst),
-        "l"(map), "r"(c0), "r"(c1), "r"(bar)
-        : "memory");
-}
-
-// K-major operand with 128-byte swizzle: rows of 128 bytes, groups of 8 rows
-// 1024 bytes apart; descriptor version 1 (sm_100), layout type 2.
-__device__ __forceinline__ uint64_t umma_desc_sw128(uint32_t smem_addr) {
-    return (uint64_t)((smem_addr & 0x3FFFFu) >> 4) | ((uint64_t)1 << 16) | ((uint64_t)(1024 >> 4) << 32) |
-           ((uint64_t)1 << 46) | ((uint64_t)2 << 61);
-}
-
-// Bounded wait for a phase of an mbarrier.  mbarrier.try_wait suspends the thread in hardware for a short,
-// system-dependent time and wakes it when the phase completes, so a poll is cheap; after a first burst the
-// thread also looks at the CTA's abort flag and sleeps briefly between polls.  The limit is TIME on the
-// global timer (the duration of a poll is not specified, so an iteration count alone bounds nothing): when
-// it runs out the CTA-wide abort flag is raised, every role leaves its loop and the kernel ends with status 4.
-constexpr unsigned long long kLgWaitLimitNs = 2000ull * 1000ull * 1000ull;
-__device__ __forceinline__ bool wait_or_abort(uint32_t bar, uint32_t parity, volatile int* abort_flag) {
-    unsigned long long t0 = 0;
-    for (uint32_t it = 0; it < (1u << 28); ++it) {
-        if (mbar_test(bar, parity)) return true;
-        if (it >= 32) {
-            if (*abort_flag) return false;
-            if ((it & 63u) == 32u) {
-                const unsigned long long now = global_timer_ns();
-                if (t0 == 0) t0 = now;
-                else if (now - t0 > kLgWaitLimitNs) break;
-            }
-            __nanosleep(64);
-        }
-    }
-    *abort_flag = 1;
-    return false;
-}
 
 // Epilogue of one 16-token slice of one output column: v = the 16 accumulators, sc = the tokens' scales
 // (or prefill coefficients ws/s), o0 = index of the first output element, live = tokens to store.

@@ -77,7 +77,7 @@ class DecoderOpsError(RuntimeError):
 
 def check(status: int):
     if status:
-        raise DecoderOpsError({1: "shape not supported", 2: "bad pointer", 3: "launch failed"}.get(status, str(status)))
+        raise DecoderOpsError({1: "shape not supported", 2: "bad pointer", 3: "launch failed", 4: "a wait inside a kernel ran out"}.get(status, str(status)))
 
 
 def load_decoder_library() -> ctypes.CDLL:
@@ -103,12 +103,15 @@ def load_decoder_library() -> ctypes.CDLL:
         fn.restype = _I
     lib.decoder_head_scratch_bytes.argtypes = []
     lib.decoder_head_scratch_bytes.restype = L
+    lib.decoder_status.argtypes = []
+    lib.decoder_status.restype = _I
     _DECODER_LIB = lib
     return lib
 
 
 DECODER_SYMBOLS = ("decoder_embed", "decoder_hyper", "decoder_rows_linear", "decoder_head_scratch_bytes",
-                   "decoder_head_argmax", "decoder_relu2", "decoder_delta", "decoder_tanh_cols", "decoder_attn")
+                   "decoder_head_argmax", "decoder_relu2", "decoder_delta", "decoder_tanh_cols", "decoder_attn",
+                   "decoder_status")
 
 
 def load_library() -> ctypes.CDLL:
