@@ -29,6 +29,21 @@ __device__ __forceinline__ float ld_cg(const float* p) { return __ldcg(p); }
 __device__ __forceinline__ float ld_cg(const bf16* p) {
     return __bfloat162float(__ushort_as_bfloat16(__ldcg(reinterpret_cast<const unsigned short*>(p))));
 }
+// the same without the conversion, for loads that are to stay in flight
+template <typename T>
+struct Raw;
+template <>
+struct Raw<float> {
+    float v;
+    __device__ __forceinline__ void load(const float* p) { v = __ldcg(p); }
+    __device__ __forceinline__ float get() const { return v; }
+};
+template <>
+struct Raw<bf16> {
+    unsigned short v;
+    __device__ __forceinline__ void load(const bf16* p) { v = __ldcg(reinterpret_cast<const unsigned short*>(p)); }
+    __device__ __forceinline__ float get() const { return __bfloat162float(__ushort_as_bfloat16(v)); }
+};
 // four neighbouring elements (16-byte aligned fp32, 8-byte aligned bf16)
 __device__ __forceinline__ float4 ld_cg4(const float* p) { return __ldcg(reinterpret_cast<const float4*>(p)); }
 __device__ __forceinline__ float4 ld_cg4(const bf16* p) {
@@ -55,6 +70,13 @@ __device__ __forceinline__ void unpack8(uint4 v, float (&f)[8]) {
 }
 
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + __expf(-z)); }
+
+// the same with the approximate reciprocal (1 ulp; 0 when the exponential overflows)
+__device__ __forceinline__ float sigmoid_fast(float z) {
+    float r;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + __expf(-z)));
+    return r;
+}
 
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll

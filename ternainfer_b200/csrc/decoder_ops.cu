@@ -88,6 +88,8 @@ static int hyper(const HyperParams& p, int pdl, void* stream) {
     return bad(DECODER_BAD_SHAPE, "hyper: 1 to 8 streams");
 }
 
+static bool quads(int n) { return n >= 4 && n <= 128 && (n & (n - 1)) == 0; }
+
 template <typename A>
 static int delta_prompt(const DeltaParams& p, int pdl, void* stream) {
     const dim3 grid((p.dv + kScanCols - 1) / kScanCols, p.H, p.B);
@@ -98,7 +100,22 @@ static int delta_prompt(const DeltaParams& p, int pdl, void* stream) {
     else rc = launch(delta_scan_kernel<A, 32>, grid, 256, ScanShape<32>::smem, pdl, stream, 1, p);
     if (rc) return rc;
     const long long units = (long long)p.B * p.T * p.H;
+    if (quads(p.dv) && p.ld % 4 == 0 && p.off_g % 4 == 0 && !misaligned(p.proj, 16) && !misaligned(p.y, 16) && !misaligned(p.norm, 16))
+        return launch(delta_finish4_kernel<A>, dim3((unsigned)((units * p.dv + 2047) / 2048)), 256, 0, pdl, stream, 1, p);
     return launch(delta_finish_kernel<A>, dim3((unsigned)((units + 7) / 8)), 256, 0, pdl, stream, 1, p);
+}
+
+template <typename A, int NR>
+static int delta_one_n(const DeltaParams& p, int dvp, int pdl, void* stream) {
+    const int words = p.dk * (p.rank / 8);
+    const bool wide = sizeof(A) == 2 && p.rank % 8 == 0 && words <= 4 * kStepThreads && !misaligned(p.w2, 16);
+    const size_t smem = ((size_t)5 * p.dk + (p.rank + 3) / 4 * 4 + std::max(kStepThreads, wide ? words : 0)) * 4;
+    const dim3 grid(p.H, p.B);
+    if constexpr (sizeof(A) == 2) {
+        if (wide && words <= kStepThreads) return launch(delta_step_kernel<A, NR, 1>, grid, kStepThreads, smem, pdl, stream, 1, p, dvp);
+        if (wide) return launch(delta_step_kernel<A, NR, 4>, grid, kStepThreads, smem, pdl, stream, 1, p, dvp);
+    }
+    return launch(delta_step_kernel<A, NR, 0>, grid, kStepThreads, smem, pdl, stream, 1, p, dvp);
 }
 
 template <typename A>
@@ -106,20 +123,16 @@ static int delta_one(const DeltaParams& p, int pdl, void* stream) {
     int dvp = 32;
     while (dvp < p.dv) dvp <<= 1;
     const int rows = (p.dk + kStepThreads / dvp - 1) / (kStepThreads / dvp);
-    const size_t smem = ((size_t)5 * p.dk + p.rank + kStepThreads) * 4;
-    const dim3 grid(p.H, p.B);
-    if (rows <= 8) return launch(delta_step_kernel<A, 8>, grid, kStepThreads, smem, pdl, stream, 1, p, dvp);
-    if (rows <= 16) return launch(delta_step_kernel<A, 16>, grid, kStepThreads, smem, pdl, stream, 1, p, dvp);
-    if (rows <= 32) return launch(delta_step_kernel<A, 32>, grid, kStepThreads, smem, pdl, stream, 1, p, dvp);
-    return launch(delta_step_kernel<A, 0>, grid, kStepThreads, smem, pdl, stream, 1, p, dvp);
+    if (rows <= 8) return delta_one_n<A, 8>(p, dvp, pdl, stream);
+    if (rows <= 32) return delta_one_n<A, 32>(p, dvp, pdl, stream);
+    return delta_one_n<A, 0>(p, dvp, pdl, stream);
 }
 
 template <int RT, int LPK>
 static int attn_one(const AttnParams& p, int pdl, void* stream) {
     const int rep = p.H / p.G, units = p.G * ((rep + RT - 1) / RT);
-    // slices of the slots: enough CTAs to fill the chip, at least 64 slots each
-    int nr = 1;
-    while (nr < 8 && units * p.B * nr * 2 <= 2 * sm_count() && p.slots >= 64 * nr * 2) nr *= 2;
+    // slices of the slots: as many CTAs as the chip holds at a time, at least 64 slots each
+    const int nr = std::max(1, std::min(std::min(8, (RT <= 4 ? 2 : 1) * sm_count() / (units * p.B)), p.slots / 64));
     return launch(sigmoid_attn_step_kernel<RT, LPK>, dim3(nr, units, p.B), 256, 0, pdl, stream, nr, p);
 }
 template <int LPK>
@@ -169,7 +182,10 @@ static int attn_tc(const AttnParams& p, void* stream) {
 template <typename A>
 static int attn_prompt(const AttnParams& p, bool tensor_cores, int pdl, void* stream) {
     const long long units = (long long)p.B * p.T * (p.H + p.G);
-    int rc = launch(head_norm_kernel<A>, dim3((unsigned)((units + 7) / 8)), 256, 0, pdl, stream, 1, p);
+    const bool vec = quads(p.dim) && p.ld % 4 == 0 && p.off_q % 4 == 0 && p.off_k == p.off_q + p.H * p.dim && !misaligned(p.proj, 16) &&
+                     !misaligned(p.q_norm, 16) && !misaligned(p.k_norm, 16);
+    int rc = vec ? launch(head_norm4_kernel<A>, dim3((unsigned)((units * p.dim + 2047) / 2048)), 256, 0, pdl, stream, 1, p)
+                 : launch(head_norm_kernel<A>, dim3((unsigned)((units + 7) / 8)), 256, 0, pdl, stream, 1, p);
     if (rc) return rc;
     rc = tensor_cores ? attn_tc(p, stream)
                       : launch(sigmoid_attn_plain_kernel<A>, dim3(p.T, p.H, p.B), 128, (size_t)(p.dim + p.vdim) * 4, pdl, stream, 1, p);
@@ -235,8 +251,8 @@ extern "C" int decoder_relu2(void* x, long long n, int dtype, int pdl, void* str
 extern "C" int decoder_delta(const decoder_delta_args* a, int dtype, int pdl, void* stream) {
     if (a->B < 1 || a->T < 1 || a->H < 1 || a->dk < 1 || a->dv < 1 || a->rank < 1 || a->dk > 256 || a->dv > 512)
         return bad(DECODER_BAD_SHAPE, "delta: 1 <= dk <= 256, 1 <= dv <= 512");
-    if (!a->proj || !a->w0 || !a->a_bias || !a->norm || !a->pos || !a->state || !a->y || (a->T > 1 ? !a->zw || !a->o : !a->w2))
-        return bad(DECODER_BAD_POINTER, "delta: null pointer");
+    if (!a->proj || !a->w0 || !a->a_bias || !a->norm || !a->pos || !a->state || !a->y || (a->T > 1 ? !a->zw || !a->o || misaligned(a->o, 16) : !a->w2))
+        return bad(DECODER_BAD_POINTER, "delta: null or misaligned pointer");
     if (a->T == 1) return dtype ? delta_one<float>(*a, pdl, stream) : delta_one<bf16>(*a, pdl, stream);
     return dtype ? delta_prompt<float>(*a, pdl, stream) : delta_prompt<bf16>(*a, pdl, stream);
 }

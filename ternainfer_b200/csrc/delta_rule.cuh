@@ -16,6 +16,7 @@
 #pragma once
 #include "decoder_common.cuh"
 #include "decoder_ops.h"
+#include "lm_head.cuh"
 
 namespace tsp {
 
@@ -246,6 +247,37 @@ __global__ void __launch_bounds__(256) delta_finish_kernel(const DeltaParams p) 
         y[c] = from_f<A>(ld_cg(o + c) * inv * p.norm[head * dv + c] * sigmoid_f(ld_cg(g + c)));
 }
 
+// The same with four neighbouring columns per lane: dv a power of two from 4 to 128, so that dv / 4 lanes share a head;
+// two units of 128 columns per warp in flight.
+template <typename A>
+__global__ void __launch_bounds__(256) delta_finish4_kernel(const DeltaParams p) {
+    griddep_launch_dependents();
+    griddep_wait();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const long long n = (long long)p.H * p.dv, total = (long long)p.B * p.T * n;
+    float4 o[2], g[2];
+    long long at[2];
+    int col[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        at[i] = (((long long)blockIdx.x * 8 + warp) * 2 + i) * 128 + lane * 4;
+        const long long e = min(at[i], total - 4), row = e / n;
+        col[i] = (int)(e - row * n);
+        o[i] = ld_cg4(p.o + e);
+        g[i] = ld_cg4(reinterpret_cast<const A*>(p.proj) + row * p.ld + p.off_g + col[i]);
+    }
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        float ss = o[i].x * o[i].x + o[i].y * o[i].y + o[i].z * o[i].z + o[i].w * o[i].w;
+        for (int d = p.dv / 8; d; d >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, d);
+        const float inv = 1.f / sqrtf(ss / (float)p.dv + p.eps);
+        const float4 w = *reinterpret_cast<const float4*>(p.norm + col[i]);
+        if (at[i] < total)
+            st4(reinterpret_cast<A*>(p.y) + at[i], make_float4(o[i].x * inv * w.x * sigmoid_fast(g[i].x), o[i].y * inv * w.y * sigmoid_fast(g[i].y),
+                                                               o[i].z * inv * w.z * sigmoid_fast(g[i].z), o[i].w * inv * w.w * sigmoid_fast(g[i].w)));
+    }
+}
+
 // t1[row][j] = tanh of the low-rank decay projection, contiguous (input of the second projection of a prompt)
 template <typename A>
 __global__ void __launch_bounds__(256) tanh_cols_kernel(const A* proj, long long ld, int off, int rank, long long rows, A* out) {
@@ -260,8 +292,10 @@ __global__ void __launch_bounds__(256) tanh_cols_kernel(const A* proj, long long
 // ------------------------------------------------------------------------------------------ one token
 constexpr int kStepThreads = 512;
 
-// NR: state rows a thread keeps in registers (dk <= NR * row groups); 0: the state is read twice instead
-template <typename A, int NR>
+// NR: state rows a thread keeps in registers (dk <= NR * row groups); 0: the state is read twice instead.
+// WIDE: rank a multiple of 8 and dk * rank / 8 words of 16 bytes of w2 (bf16) are at most WIDE per thread: they are
+// requested before the wait for the projections.
+template <typename A, int NR, int WIDE>
 __global__ void __launch_bounds__(kStepThreads) delta_step_kernel(const DeltaParams p, const int dvp) {
     extern __shared__ __align__(16) float step_smem[];
     __shared__ float red[32];
@@ -271,15 +305,21 @@ __global__ void __launch_bounds__(kStepThreads) delta_step_kernel(const DeltaPar
     const int RG = kStepThreads / dvp;                      // row groups; dvp a power of two >= dv
     float* u_s = step_smem;
     float *w_s = u_s + dk, *au_s = w_s + dk, *k_s = au_s + dk, *r_s = k_s + dk, *t1_s = r_s + dk;
-    float* part = t1_s + rank;                              // [RG][dvp]
+    float* part = t1_s + (rank + 3) / 4 * 4;                // [RG][dvp], and the decay's partial sums [dk][rank / 8]
     griddep_launch_dependents();
     const A* w2 = reinterpret_cast<const A*>(p.w2) + (size_t)head * dk * rank;
-    for (size_t i = (size_t)tid * 128; i < (size_t)dk * rank * sizeof(A); i += (size_t)kStepThreads * 128)
-        asm volatile("prefetch.global.L2 [%0];" ::"l"(reinterpret_cast<const char*>(w2) + i));
+    const int per = rank / 8, words = dk * per;             // (WIDE) a word = 8 ranks of one channel
+    uint4 wv[WIDE > 0 ? WIDE : 1];
+    if constexpr (WIDE > 0) {
+#pragma unroll
+        for (int i = 0; i < WIDE; ++i) {
+            const int e = tid + i * kStepThreads;
+            wv[i] = e < words ? ldg_stream_128(w2 + (size_t)e * 8) : make_uint4(0, 0, 0, 0);
+        }
+    }
     griddep_wait();
     const A* row = reinterpret_cast<const A*>(p.proj) + (size_t)b * p.ld;
     float* st = p.state + ((size_t)b * p.H + head) * dk * dv;
-    const bool fresh = p.pos[0] == 0;
     const int col = tid & (dvp - 1), rg = tid / dvp;
     const bool live = col < dv;
     float s[NR > 0 ? NR : 1];
@@ -287,29 +327,53 @@ __global__ void __launch_bounds__(kStepThreads) delta_step_kernel(const DeltaPar
 #pragma unroll
         for (int i = 0; i < NR; ++i) {
             const int k = rg + i * RG;
-            s[i] = (!fresh && live && k < dk) ? ld_cg(st + (size_t)k * dv + col) : 0.f;
+            s[i] = (live && k < dk) ? ld_cg(st + (size_t)k * dv + col) : 0.f;
         }
     }
+    const bool fresh = p.pos[0] == 0;
     const float v = live ? ld_cg(row + p.off_v + head * dv + col) : 0.f;
+    const float gate = live ? ld_cg(row + p.off_g + head * dv + col) : 0.f;
     float ss = 0.f;
     for (int c = tid; c < dk; c += kStepThreads) {
         const float k = ld_cg(row + p.off_k + head * dk + c);
         k_s[c] = k, r_s[c] = ld_cg(row + p.off_r + head * dk + c);
+        au_s[c] = sigmoid_f(ld_cg(row + p.off_a + head * dk + c) + p.a_bias[head * dk + c]);
         ss = fmaf(k, k, ss);
     }
     for (int c = tid; c < rank; c += kStepThreads) t1_s[c] = tanhf(ld_cg(row + p.off_w1 + c));
     const float inv = 1.f / sqrtf(block_sum(ss, red) + 1e-6f);
-    // decay: one warp per channel, lanes over the rank
-    for (int c = warp; c < dk; c += nw) {
+    if constexpr (WIDE > 0) {
+#pragma unroll
+        for (int i = 0; i < WIDE; ++i) {
+            const int e = tid + i * kStepThreads;
+            if (e < words) {
+                float f[8], z = 0.f;
+                unpack8(wv[i], f);
+                const float* t = t1_s + (e % per) * 8;
+#pragma unroll
+                for (int j = 0; j < 8; ++j) z = fmaf(f[j], t[j], z);
+                part[e] = z;
+            }
+        }
+        __syncthreads();
+    }
+    for (int c = WIDE > 0 ? tid : warp; c < dk; c += WIDE > 0 ? kStepThreads : nw) {
         float z = 0.f;
-        for (int j = lane; j < rank; j += 32) z = fmaf(to_f(w2[(size_t)c * rank + j]), t1_s[j], z);
-        z = warp_sum(z);
-        if (lane == 0) {
-            const float a = sigmoid_f(ld_cg(row + p.off_a + head * dk + c) + p.a_bias[head * dk + c]);
+        if constexpr (WIDE > 0) {
+            for (int j = 0; j < per; ++j) z += part[c * per + j];
+        } else {                                            // one warp per channel, lanes over the rank
+            for (int j = lane; j < rank; j += 32) z = fmaf(to_f(w2[(size_t)c * rank + j]), t1_s[j], z);
+            z = warp_sum(z);
+        }
+        if (WIDE > 0 || lane == 0) {
             const float u = k_s[c] * inv;
-            u_s[c] = u, au_s[c] = a * u;
+            u_s[c] = u, au_s[c] *= u;
             w_s[c] = __expf(-kDecayScale * sigmoid_f(z + p.w0[head * dk + c]));
         }
+    }
+    if (fresh) {
+#pragma unroll
+        for (int i = 0; i < (NR > 0 ? NR : 1); ++i) s[i] = 0.f;
     }
     __syncthreads();
     float seen = 0.f;
@@ -351,8 +415,7 @@ __global__ void __launch_bounds__(kStepThreads) delta_step_kernel(const DeltaPar
     __syncthreads();                                        // red is reused
     const float on = 1.f / sqrtf(block_sum(rg == 0 && live ? o * o : 0.f, red) / (float)dv + p.eps);
     if (rg == 0 && live) {
-        const float g = sigmoid_f(ld_cg(row + p.off_g + head * dv + col));
-        reinterpret_cast<A*>(p.y)[(size_t)b * p.H * dv + head * dv + col] = from_f<A>(o * on * p.norm[head * dv + col] * g);
+        reinterpret_cast<A*>(p.y)[(size_t)b * p.H * dv + head * dv + col] = from_f<A>(o * on * p.norm[head * dv + col] * sigmoid_f(gate));
     }
 }
 

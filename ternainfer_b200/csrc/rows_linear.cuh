@@ -13,7 +13,7 @@
 namespace tsp {
 
 constexpr int kRowsWarps = 8;
-constexpr int kRowsPre = 8;   // k-steps of 32 whose weights are in flight per warp
+constexpr int kRowsPre = 6;   // k-steps of 32 whose weights are in flight per warp: what two CTAs per SM have registers for
 
 struct RowsLinearParams {
     const bf16* x;     // [M][K]
@@ -24,7 +24,7 @@ struct RowsLinearParams {
 };
 
 template <typename O>
-__global__ void __launch_bounds__(kRowsWarps * 32) rows_linear_kernel(const RowsLinearParams p) {
+__global__ void __launch_bounds__(kRowsWarps * 32, 2) rows_linear_kernel(const RowsLinearParams p) {
     __shared__ float part[kRowsWarps][16][9];
     griddep_launch_dependents();
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;

@@ -38,6 +38,37 @@ __global__ void __launch_bounds__(256) head_norm_kernel(const AttnParams p) {
     for (int c = lane; c < dim; c += 32) x[c] = from_f<A>(ld_cg(x + c) * inv * w[c]);
 }
 
+// The same with four neighbouring channels per lane: dim a power of two from 4 to 128 (dim / 4 lanes share a head), q
+// and k side by side; two units of 128 channels per warp in flight.
+template <typename A>
+__global__ void __launch_bounds__(256) head_norm4_kernel(const AttnParams p) {
+    griddep_launch_dependents();
+    griddep_wait();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const long long n = (long long)(p.H + p.G) * p.dim, total = (long long)p.B * p.T * n;
+    float4 x[2];
+    long long at[2];
+    A* dst[2];
+    const float* w[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        at[i] = (((long long)blockIdx.x * 8 + warp) * 2 + i) * 128 + lane * 4;
+        const long long e = min(at[i], total - 4), row = e / n;
+        const int c = (int)(e - row * n);
+        dst[i] = reinterpret_cast<A*>(p.proj) + row * p.ld + p.off_q + c;
+        w[i] = (c < p.H * p.dim ? p.q_norm : p.k_norm) + (c & (p.dim - 1));
+        x[i] = ld_cg4(dst[i]);
+    }
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        float ss = x[i].x * x[i].x + x[i].y * x[i].y + x[i].z * x[i].z + x[i].w * x[i].w;
+        for (int d = p.dim / 8; d; d >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, d);
+        const float inv = 1.f / sqrtf(ss / (float)p.dim + p.eps);
+        const float4 g = *reinterpret_cast<const float4*>(w[i]);
+        if (at[i] < total) st4(dst[i], make_float4(x[i].x * inv * g.x, x[i].y * inv * g.y, x[i].z * inv * g.z, x[i].w * inv * g.w));
+    }
+}
+
 // Any type, any sizes: one CTA per query and head, 128 keys at a time.  Queries and keys already normalised.
 template <typename A>
 __global__ void __launch_bounds__(128) sigmoid_attn_plain_kernel(const AttnParams p) {
@@ -97,11 +128,13 @@ __global__ void __launch_bounds__(128) attn_cache_store_kernel(const AttnParams 
     const size_t slot = (size_t)(i % p.chunk);
     if (slot >= (size_t)p.slots) return;
     const A* row = reinterpret_cast<const A*>(p.proj) + ((size_t)b * p.T + t) * p.ld;
-    for (int g = 0; g < p.G; ++g) {
-        A* k = reinterpret_cast<A*>(p.ck) + (((size_t)b * p.G + g) * p.slots + slot) * p.dim;
-        A* v = reinterpret_cast<A*>(p.cv) + (((size_t)b * p.G + g) * p.slots + slot) * p.vdim;
-        for (int c = threadIdx.x; c < p.dim; c += blockDim.x) k[c] = from_f<A>(ld_cg(row + p.off_k + g * p.dim + c));
-        for (int c = threadIdx.x; c < p.vdim; c += blockDim.x) v[c] = from_f<A>(ld_cg(row + p.off_v + g * p.vdim + c));
+    for (int e = threadIdx.x; e < p.G * p.dim; e += blockDim.x) {
+        const int g = e / p.dim, c = e - g * p.dim;
+        reinterpret_cast<A*>(p.ck)[(((size_t)b * p.G + g) * p.slots + slot) * p.dim + c] = from_f<A>(ld_cg(row + p.off_k + e));
+    }
+    for (int e = threadIdx.x; e < p.G * p.vdim; e += blockDim.x) {
+        const int g = e / p.vdim, c = e - g * p.vdim;
+        reinterpret_cast<A*>(p.cv)[(((size_t)b * p.G + g) * p.slots + slot) * p.vdim + c] = from_f<A>(ld_cg(row + p.off_v + e));
     }
 }
 
@@ -111,9 +144,16 @@ __global__ void __launch_bounds__(128) attn_cache_store_kernel(const AttnParams 
 // and RT of its query heads: each CTA takes a slice of the slots, a key being handled by LPK lanes with eight
 // channels each; partial outputs (plain sums, as the weights are not normalised) meet in distributed shared
 // memory in a fixed order.
+//
+// A warp has U keys per lane group in flight.  Their RT * U scores are summed over the LPK lanes by a transposing
+// butterfly that leaves each score in one lane (or a few), where its weight is computed once; the weights are then
+// handed back to all lanes for the values' sum.
 template <int RT, int LPK>
-__global__ void __launch_bounds__(256) sigmoid_attn_step_kernel(const AttnParams p) {
-    constexpr int KPW = 32 / LPK, VD = 8 * LPK, U = 4;       // keys per warp at a time, padded width, unroll
+__global__ void __launch_bounds__(256, RT <= 4 ? 2 : 1) sigmoid_attn_step_kernel(const AttnParams p) {
+    constexpr int KPW = 32 / LPK, VD = 8 * LPK;              // keys per warp at a time, padded width
+    constexpr int U = RT <= 2 ? 8 : RT <= 4 ? 4 : 2, NV = RT * U;
+    constexpr int LL = LPK == 4 ? 2 : LPK == 8 ? 3 : LPK == 16 ? 4 : 5, LN = NV == 8 ? 3 : 4;
+    constexpr int EX = LL < LN ? LL : LN, REM = NV >> EX;    // exchange levels of the butterfly, scores left per lane
     __shared__ __align__(16) float q_s[RT][VD];
     __shared__ __align__(16) float k_s[VD];
     __shared__ __align__(16) float v_s[VD];
@@ -130,7 +170,7 @@ __global__ void __launch_bounds__(256) sigmoid_attn_step_kernel(const AttnParams
     bf16* cv = reinterpret_cast<bf16*>(p.cv) + ((size_t)b * p.G + g) * p.slots * vdim;
     griddep_wait();
     const bf16* row = reinterpret_cast<const bf16*>(p.proj) + (size_t)b * p.ld;
-    const int cur = (int)(p.pos[0] % p.chunk);               // slot of this token = number of earlier visible keys
+    const int cur = (int)((unsigned)p.pos[0] % (unsigned)p.chunk);   // slot of this token = number of earlier visible keys
     const bool writer = rank == 0 && blockIdx.y % hgroups == 0 && cur < p.slots;
 
     for (int e = warp; e < RT + 2; e += 8) {
@@ -171,50 +211,88 @@ __global__ void __launch_bounds__(256) sigmoid_attn_step_kernel(const AttnParams
     __syncthreads();
 
     const int sub = lane / LPK, c8 = (lane % LPK) * 8;
-    float q[RT][8], acc[RT][8], slope[RT], bias[RT];
+    const int v0 = ((lane % LPK) >> (LL - EX)) * REM;        // first of the scores whose weights this lane computes
+    float q[RT][8], acc[RT][8], slope[REM], bias[REM];
 #pragma unroll
-    for (int r = 0; r < RT; ++r) {
-        slope[r] = r < hn ? p.slope[h0 + r] : 0.f;
-        bias[r] = r < hn ? p.bias[h0 + r] : 0.f;
+    for (int i = 0; i < REM; ++i) {
+        const int r = (v0 + i) / U;
+        slope[i] = r < hn ? p.slope[h0 + r] : 0.f;
+        bias[i] = r < hn ? p.bias[h0 + r] : 0.f;
+    }
+#pragma unroll
+    for (int r = 0; r < RT; ++r)
 #pragma unroll
         for (int c = 0; c < 8; ++c) q[r][c] = q_s[r][c8 + c], acc[r][c] = 0.f;
-    }
-    auto use = [&](const float (&k)[8], const float (&v)[8], int j, bool on) {
+    // scores of keys j0 + u * KPW + sub for u < U (those below hi count), weights, weighted values
+    auto use = [&](const uint4 (&kv)[U], const uint4 (&vv)[U], int j0, int hi) {
+        float s[NV];
 #pragma unroll
-        for (int r = 0; r < RT; ++r) {
-            float s = 0.f;
+        for (int u = 0; u < U; ++u) {
+            float k[8];
+            unpack8(kv[u], k);
 #pragma unroll
-            for (int c = 0; c < 8; ++c) s = fmaf(q[r][c], k[c], s);
+            for (int r = 0; r < RT; ++r) {
+                float d = q[r][0] * k[0];
 #pragma unroll
-            for (int d = LPK / 2; d; d >>= 1) s += __shfl_xor_sync(0xffffffffu, s, d);
-            const float w = on ? sigmoid_f(s - slope[r] * (float)(cur - j) + bias[r]) : 0.f;
+                for (int c = 1; c < 8; ++c) d = fmaf(q[r][c], k[c], d);
+                s[r * U + u] = d;
+            }
+        }
 #pragma unroll
-            for (int c = 0; c < 8; ++c) acc[r][c] = fmaf(w, v[c], acc[r][c]);
+        for (int l = 0; l < LL; ++l) {
+            const int d = LPK >> (l + 1), n = NV >> (l + 1);
+            if (l < EX) {
+#pragma unroll
+                for (int i = 0; i < n; ++i) {
+                    const bool up = lane & d;
+                    const float keep = up ? s[i + n] : s[i], give = up ? s[i] : s[i + n];
+                    s[i] = keep + __shfl_xor_sync(0xffffffffu, give, d);
+                }
+            } else {
+                s[0] += __shfl_xor_sync(0xffffffffu, s[0], d);
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < REM; ++i) {
+            const int j = j0 + (v0 + i) % U * KPW + sub;
+            s[i] = j < hi ? sigmoid_fast(s[i] - slope[i] * (float)(cur - j) + bias[i]) : 0.f;
+        }
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+            float v[8];
+            unpack8(vv[u], v);
+#pragma unroll
+            for (int r = 0; r < RT; ++r) {
+                const int n = r * U + u;
+                const float w = __shfl_sync(0xffffffffu, s[n % REM], sub * LPK + ((n / REM) << (LL - EX)));
+#pragma unroll
+                for (int c = 0; c < 8; ++c) acc[r][c] = fmaf(w, v[c], acc[r][c]);
+            }
         }
     };
     const int lo = (int)((long long)cur * rank / nr), hi = (int)((long long)cur * (rank + 1) / nr);
     const bool kin = c8 < dim, vin = c8 < vdim;
+    const uint4 zero = make_uint4(0, 0, 0, 0);
     for (int j0 = lo + warp * KPW * U; j0 < hi; j0 += 8 * KPW * U) {
         uint4 kv[U], vv[U];
 #pragma unroll
         for (int u = 0; u < U; ++u) {
             const int j = j0 + u * KPW + sub;
-            kv[u] = (j < hi && kin) ? ld_cg_128(ck + (size_t)j * dim + c8) : make_uint4(0, 0, 0, 0);
-            vv[u] = (j < hi && vin) ? ld_cg_128(cv + (size_t)j * vdim + c8) : make_uint4(0, 0, 0, 0);
+            kv[u] = (j < hi && kin) ? ld_cg_128(ck + (size_t)j * dim + c8) : zero;
+            vv[u] = (j < hi && vin) ? ld_cg_128(cv + (size_t)j * vdim + c8) : zero;
         }
-#pragma unroll
-        for (int u = 0; u < U; ++u) {
-            const int j = j0 + u * KPW + sub;
-            float k[8], v[8];
-            unpack8(kv[u], k), unpack8(vv[u], v);
-            use(k, v, j, j < hi);
-        }
+        use(kv, vv, j0, hi);
     }
-    if (rank == nr - 1 && warp == 7) {                       // the token itself
-        float k[8], v[8];
+    if (rank == nr - 1 && warp == 7) {                       // the token itself: bf16 values, so packing loses nothing
+        uint4 kv[U], vv[U];
 #pragma unroll
-        for (int c = 0; c < 8; ++c) k[c] = k_s[c8 + c], v[c] = v_s[c8 + c];
-        use(k, v, cur, sub == 0);
+        for (int u = 0; u < U; ++u) kv[u] = vv[u] = zero;
+        if (sub == 0) {
+            const float *k = k_s + c8, *v = v_s + c8;
+            kv[0] = make_uint4(pack_bf16(k[0], k[1]), pack_bf16(k[2], k[3]), pack_bf16(k[4], k[5]), pack_bf16(k[6], k[7]));
+            vv[0] = make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
+        }
+        use(kv, vv, cur, cur + 1);
     }
 #pragma unroll
     for (int r = 0; r < RT; ++r)
