@@ -1022,6 +1022,235 @@ def run_decode_arm(args):
     print(json.dumps(line), flush=True)
 
 
+# ----------------------------------------------------------------------------
+# Kepovik workload: the decoder of ternainfer_b200/kepovik.py beside the ternary
+# model of equal width, feed-forward, heads and layer count (the closest one the
+# framework has), whole models and kernel by kernel.
+# ----------------------------------------------------------------------------
+
+KEPOVIK_SIZES = {   # width, feed-forward, attention heads, kv heads, head dim, delta heads, delta dim, layers
+    "2560": (2560, 6912, 20, 5, 128, 40, 64, 30),
+    "4096": (4096, 14336, 32, 8, 128, 64, 64, 8),
+}
+KEPOVIK_VOCAB, KEPOVIK_CHUNK, KEPOVIK_RANK, KEPOVIK_STREAMS = 128256, 2048, 64, 4
+
+
+def kepovik_config(size):
+    """Delta and attention layers in turn, a feed-forward in every layer."""
+    width, ff, heads, kv, dim, dh, dd, layers = KEPOVIK_SIZES[size]
+    mlp = {"kind": "dense", "ff": ff}
+    delta = {"type": "general_delta", "mixer": {"heads": dh, "dim": dd}, "mlp": mlp}
+    attn = {"type": "attention", "mlp": mlp, "mixer": {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": dim,
+                                                       "mask": {"size": KEPOVIK_CHUNK}, "scale": dim ** -0.5}}
+    return {"architecture": "Kepovik", "vocab": KEPOVIK_VOCAB, "width": width, "streams": KEPOVIK_STREAMS, "norm": {"eps": 1e-5},
+            "residual_mult": 0.5, "layers": [delta if i % 2 == 0 else attn for i in range(layers)],
+            "embedding": {"bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 17}}}
+
+
+def kepovik_model(size, max_len, seed):
+    import torch
+    from ternainfer_b200.kepovik import Kepovik, parse_config, random_checkpoint
+    args = parse_config(kepovik_config(size))
+    return Kepovik(args, random_checkpoint(args, KEPOVIK_RANK, seed), max_seq_len=max_len, dtype=torch.bfloat16).cuda()
+
+
+def ternary_model(size, max_len, seed):
+    from ternainfer_b200.generate import build_random_model
+    from ternainfer_b200.linear import reserve_workspace
+    from ternainfer_b200.model import ModelArgs
+    width, ff, heads, kv, dim, _, _, layers = KEPOVIK_SIZES[size]
+    reserve_workspace(2 * ff * width)
+    return build_random_model(ModelArgs(dim=width, n_layers=layers, n_heads=heads, n_kv_heads=kv, ffn_dim=ff,
+                                        vocab_size=KEPOVIK_VOCAB, fused_glue=True), max_len, seed)[0]
+
+
+def graph_us(torch, calls, steps, warmup):
+    """Device time per call of a list of calls captured in one graph (CUDA events, `steps` replays)."""
+    with torch.inference_mode():
+        for c in calls:
+            c()
+        torch.cuda.synchronize()
+        g = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(g):
+            for c in calls:
+                c()
+        for _ in range(warmup):
+            g.replay()
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        a.record()
+        for _ in range(steps):
+            g.replay()
+        b.record()
+        torch.cuda.synchronize()
+    return a.elapsed_time(b) * 1e3 / (steps * len(calls))
+
+
+def model_speed(torch, build, size, args):
+    """Prompt and decode tokens/s of a model through FastGen's captured graphs."""
+    from ternainfer_b200.generate import FastGen, GenArgs
+    out = {}
+    for P, B in ((512, 1), (2048, 1), (512, 8)):
+        model = build(size, P + 128, args.seed)
+        gen = FastGen(model, GenArgs(128, B, P, True))
+        g = torch.Generator(device="cuda").manual_seed(args.seed + 1)
+        gen.generate(torch.randint(0, KEPOVIK_VOCAB, (B, P), generator=g, device="cuda"))
+        gen._pos.fill_(P + 64)
+        ev = [torch.cuda.Event(enable_timing=True) for _ in range(3)]
+        n_pre, n_dec = max(3, args.steps // 10), args.steps
+        for _ in range(args.warmup):
+            gen._prefill_graph.replay()
+            gen._decode_graph.replay()
+        torch.cuda.synchronize()
+        ev[0].record()
+        for _ in range(n_pre):
+            gen._prefill_graph.replay()
+        ev[1].record()
+        for _ in range(n_dec):
+            gen._decode_graph.replay()
+        ev[2].record()
+        torch.cuda.synchronize()
+        pre, dec = ev[0].elapsed_time(ev[1]) / n_pre, ev[1].elapsed_time(ev[2]) / n_dec
+        out[f"prompt{P}_batch{B}"] = {"prefill_ms": pre, "prefill_tokens_per_s": 1e3 * P * B / pre, "decode_ms": dec,
+                                      "decode_tokens_per_s": 1e3 * B / dec}
+        del gen, model
+        torch.cuda.empty_cache()
+    return out
+
+
+def kepovik_kernels(torch, size, args):
+    """Every kernel of both models at this size: microseconds, algorithmic bytes and matrix FLOPs, and the fraction of the
+    larger of the two bounds (measured copy rate, measured bf16 GEMM rate; the int8 GEMM against the latter too)."""
+    from ternainfer_b200 import decoder_ops as ops
+    from ternainfer_b200.linear import lm_head_argmax, rmsnorm_quant
+    width, ff, heads, kv, dim, dh, dd, _ = KEPOVIK_SIZES[size]
+    peak, kind = measured_peak()
+    try:
+        tf = float(json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json")))["bf16_tflops"])
+    except Exception:
+        tf = 1590.0
+    S, V, bf, dev = KEPOVIK_STREAMS, KEPOVIK_VOCAB, torch.bfloat16, "cuda"
+    g = torch.Generator(device=dev).manual_seed(args.seed)
+    rnd = lambda *shape, dtype=bf, scale=1.0: (scale * torch.randn(shape, generator=g, device=dev)).to(dtype)
+    out = {"peaks": {"hbm_gbs": peak, "bf16_tflops": tf, "kind": kind}, "kepovik": {}, "ternary": {}}
+    full = 160e6                                       # more than the L2
+
+    def put(model, name, calls, nbytes, flops=0.0):
+        us = graph_us(torch, calls, max(5, args.steps // 5), args.warmup)
+        bound = max(nbytes / peak / 1e3, flops / tf / 1e6)
+        out[model][name] = {"us": us, "bytes": nbytes, "flops": flops, "bound_us": bound, "frac": bound / us}
+        torch.cuda.empty_cache()
+
+    def copies(nbytes):
+        return max(2, min(400, int(full / nbytes) + 1))
+
+    nd, na = 5 * dh * dd + KEPOVIK_RANK, 2 * heads * dim + 2 * kv * dim
+    off_d = {n: i * dh * dd for i, n in enumerate(("r", "k", "v", "a", "g", "w1"))}
+    off_a = {"q": 0, "k": heads * dim, "v": (heads + kv) * dim, "g": (heads + 2 * kv) * dim}
+    f32 = lambda *shape: rnd(*shape, dtype=torch.float32, scale=0.3)
+    for B in (1, 8):
+        tag, at = f"decode_batch{B}", torch.tensor([KEPOVIK_CHUNK - 1], device=dev)
+        for name, N, K, relu2 in (("delta_in", nd, width, False), ("mixer_out", width, dh * dd, False), ("attn_in", na, width, False),
+                                  ("ff_up_relu2", ff, width, True), ("ff_down", width, ff, False)):
+            nb = 2.0 * (N * K + B * (N + K))
+            x, ws = rnd(B, K), [rnd(N, K, scale=K ** -0.5) for _ in range(copies(nb))]
+            put("kepovik", f"{tag}/linear_{name}", [lambda w=w: ops.linear(x, w, relu2=relu2, step=True) for w in ws], nb, 2.0 * B * N * K)
+            del ws
+        xs, y, h1, w1 = rnd(B, S, width, dtype=torch.float32), rnd(B, width), f32(S), f32(width)
+        mix = torch.eye(S, device=dev)
+        put("kepovik", f"{tag}/streams_norm", [lambda: ops.hyper_norm(xs, w1, 1e-5, bf, w_in=h1, weight_offset=1.0, y=y, mix=mix, w_out=h1,
+                                                                      step=True)] * 20, B * width * (8.0 * S + 4))
+        nb = B * dh * dd * dd * 8.0 + 2.0 * dh * dd * KEPOVIK_RANK + 12.0 * B * dh * dd
+        st = [torch.zeros((B, dh, dd, dd), device=dev) for _ in range(copies(nb))]
+        z, w2, v1 = rnd(B, nd), rnd(dh * dd, KEPOVIK_RANK, scale=0.1), f32(dh * dd)
+        put("kepovik", f"{tag}/delta_step", [lambda s=s: ops.delta_rule(z, off_d, w2, v1, v1, v1, s, at, 1, 1e-5, step=True) for s in st], nb)
+        del st
+        nb = 4.0 * B * kv * KEPOVIK_CHUNK * dim
+        cc = [(rnd(B, kv, KEPOVIK_CHUNK, dim), rnd(B, kv, KEPOVIK_CHUNK, dim)) for _ in range(copies(nb))]
+        z, qn, hb = rnd(B, na), f32(dim), f32(heads) - 4
+        put("kepovik", f"{tag}/attention_2048", [lambda c=c: ops.sigmoid_attention(z, off_a, qn, qn, hb, hb, c, at, 1, heads, KEPOVIK_CHUNK,
+                                                                                   dim ** -0.5, 1e-5, step=True) for c in cc], nb)
+        del cc
+        hd, W = rnd(B, width), rnd(V, width, scale=width ** -0.5)
+        put("kepovik", f"{tag}/output_head", [lambda: ops.output_argmax(hd, W)], 2.0 * V * width)
+        del W
+    T = 2048
+    pos = torch.arange(T, device=dev)
+    xs = [rnd(T, S, width, dtype=torch.float32) for _ in range(3)]
+    y = rnd(T, width)
+    put("kepovik", "prefill2048/streams_norm", [lambda x=x: ops.hyper_norm(x, w1, 1e-5, bf, w_in=h1, weight_offset=1.0, y=y, mix=mix, w_out=h1)
+                                               for x in xs], T * width * (8.0 * S + 4))
+    del xs
+    zs, state = [rnd(T, nd) for _ in range(3)], torch.zeros((1, dh, dd, dd), device=dev)
+    put("kepovik", "prefill2048/delta_rule", [lambda z=z: ops.delta_rule(z, off_d, w2, v1, v1, v1, state, pos, T, 1e-5) for z in zs],
+        2.0 * T * (nd + dh * dd))
+    out["kepovik"]["prefill2048/delta_rule"]["fp32_fma"] = 5.0 * T * dh * dd * dd
+    zs, cc = [rnd(T, na) for _ in range(5)], (rnd(1, kv, T, dim), rnd(1, kv, T, dim))
+    att = 2.0 * T * (T + 1) * heads * dim
+    put("kepovik", "prefill2048/attention", [lambda z=z: ops.sigmoid_attention(z, off_a, qn, qn, hb, hb, cc, pos, T, heads, KEPOVIK_CHUNK,
+                                                                               dim ** -0.5, 1e-5) for z in zs], 2.0 * T * (na + heads * dim), att)
+    x, ws = rnd(T, width), [rnd(ff, width, scale=width ** -0.5) for _ in range(copies(2.0 * ff * width))]
+    put("kepovik", "prefill2048/linear_ff_up_relu2", [lambda w=w: ops.linear(x, w, relu2=True) for w in ws],
+        2.0 * (T * (width + ff) + ff * width), 2.0 * T * ff * width)
+    put("kepovik", "prefill2048/linear_ff_up", [lambda w=w: ops.linear(x, w) for w in ws], 2.0 * (T * (width + ff) + ff * width),
+        2.0 * T * ff * width)
+    del zs, ws
+
+    # the ternary model's kernels
+    model = ternary_model(size, T, args.seed)
+    from flash_attn import flash_attn_with_kvcache
+    L, lay = model.layers, list(model.layers)
+    comp = lambda m: sum(t.numel() * t.element_size() for t in (m.weight_compressed_val, m.weight_TileOffsets_global,
+                                                                m.weight_TileOffsets_median, m.weight_bitmap))
+    qkv = (heads + 2 * kv) * dim
+    for B, tag in ((1, "decode_batch1"), (8, "decode_batch8"), (T, "prefill2048")):
+        for name, pick in (("wqkv", lambda l: l.attention.wqkv), ("wo", lambda l: l.attention.wo), ("w13", lambda l: l.feed_forward.w13),
+                           ("w2", lambda l: l.feed_forward.w2)):
+            N, K = pick(L[0]).out_features, pick(L[0]).in_features
+            xq, sc = torch.randint(-127, 128, (B, K), dtype=torch.int8, device=dev), torch.ones((B, 1), dtype=bf, device=dev)
+            put("ternary", f"{tag}/linear_{name}", [lambda l=l: pick(l).forward_quantized(xq, sc) for l in lay],
+                comp(pick(L[0])) + B * (K + 2.0 * N), 2.0 * B * N * K)
+        x = rnd(B, width)
+        nw = rnd(width)
+        put("ternary", f"{tag}/norm_quant", [lambda: rmsnorm_quant(x, nw, 1e-5)] * 10, 3.0 * B * width)
+        nb_b, t_q = (B, 1) if B <= 8 else (1, B)
+        q = [rnd(nb_b, t_q, heads, dim) for _ in range(3)]
+        k1 = rnd(nb_b, t_q, kv, dim)
+        nb = 4.0 * nb_b * kv * T * dim
+        cc = [(rnd(nb_b, T, kv, dim), rnd(nb_b, T, kv, dim)) for _ in range(copies(nb))]
+        seen = torch.full((nb_b,), T - t_q, dtype=torch.int32, device=dev)
+        tabs = rnd(T, dim // 2)
+        put("ternary", f"{tag}/attention_2048", [lambda i=i, c=c: flash_attn_with_kvcache(
+            q[i % 3], c[0], c[1], k=k1, v=k1, rotary_cos=tabs, rotary_sin=tabs, cache_seqlens=seen, causal=True, rotary_interleaved=True)
+            for i, c in enumerate(cc[:60])], nb if t_q == 1 else 2.0 * T * (qkv + heads * dim), 0.0 if t_q == 1 else att)
+        del cc, q
+        if B <= 8:
+            hd = rnd(B, width)
+            put("ternary", f"{tag}/output_head", [lambda: lm_head_argmax(hd, model.tok_embeddings.weight, False, True)], 2.0 * V * width)
+    return out
+
+
+def run_kepovik_arm(args):
+    import torch
+    torch.cuda.set_device(0)
+    sampler = ClockSampler(0)
+    sampler.start()
+    res = {}
+    for size in KEPOVIK_SIZES:
+        res[size] = {"layers": KEPOVIK_SIZES[size][-1], "kepovik": model_speed(torch, kepovik_model, size, args),
+                     "ternary": model_speed(torch, ternary_model, size, args), "kernels": kepovik_kernels(torch, size, args)}
+    clocks = sampler.stop()
+    best = res["2560"]["kepovik"]["prompt512_batch1"]
+    line = {"metric": "kepovik_decode_tokens_per_s", "value": best["decode_tokens_per_s"], "unit": "tokens/s", "n_gpus": 1,
+            "steps": args.steps, "warmup": args.warmup, "ms_per_step": best["decode_ms"], "higher_is_better": True, "scaling": "weak",
+            "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
+            "config": {"workload": "kepovik_2560_30_layers_prompt512_batch1", "vocab": KEPOVIK_VOCAB, "chunk": KEPOVIK_CHUNK,
+                       "decay_rank": KEPOVIK_RANK, "streams": KEPOVIK_STREAMS, "seed": args.seed,
+                       "l2_policy": "weights, states and caches larger than L2 in rotation; decode activations stay in L2"},
+            "sizes": res, "clocks": clocks}
+    print(json.dumps(line), flush=True)
+
+
 def _finish(world):
     """Leave without tearing NCCL down: destroying a process group while CUDA
     graphs that hold NCCL kernels are alive blocks at exit, so every rank meets
@@ -1046,7 +1275,7 @@ def main():
     ap.add_argument("--tokens", type=int, default=8)
     ap.add_argument("--layers", type=int, default=30)
     ap.add_argument("--seed", type=int, default=1234)
-    ap.add_argument("--workload", default="sweep", choices=["sweep", "tp", "decode", "list", "head", "prefill"])
+    ap.add_argument("--workload", default="sweep", choices=["sweep", "tp", "decode", "list", "head", "prefill", "kepovik"])
     ap.add_argument("--unfused", action="store_true", help="decode workload: plain torch glue between the linears")
     ap.add_argument("--tp_mode", default="single", choices=["single", "fused", "exact"])
     ap.add_argument("--no_graph", action="store_true", help="tp workload: launch eagerly instead of replaying a CUDA graph")
@@ -1061,6 +1290,8 @@ def main():
         run_tp_arm(args)
     elif args.workload == "decode":
         run_decode_arm(args)
+    elif args.workload == "kepovik":
+        run_kepovik_arm(args)
     elif args.workload in ("list", "head", "prefill"):
         run_single_leg(args)
     else:

@@ -190,7 +190,7 @@ static int attn_prompt(const AttnParams& p, bool tensor_cores, int pdl, void* st
     rc = tensor_cores ? attn_tc(p, stream)
                       : launch(sigmoid_attn_plain_kernel<A>, dim3(p.T, p.H, p.B), 128, (size_t)(p.dim + p.vdim) * 4, pdl, stream, 1, p);
     if (rc) return rc;
-    return launch(attn_cache_store_kernel<A>, dim3(std::min(p.T, p.slots), p.B), 128, 0, pdl, stream, 1, p);
+    return launch(attn_cache_store_kernel<A>, dim3(std::min(p.T, p.slots), p.B, p.G), 128, 0, pdl, stream, 1, p);
 }
 
 }  // namespace tsp

@@ -128,14 +128,11 @@ __global__ void __launch_bounds__(128) attn_cache_store_kernel(const AttnParams 
     const size_t slot = (size_t)(i % p.chunk);
     if (slot >= (size_t)p.slots) return;
     const A* row = reinterpret_cast<const A*>(p.proj) + ((size_t)b * p.T + t) * p.ld;
-    for (int e = threadIdx.x; e < p.G * p.dim; e += blockDim.x) {
-        const int g = e / p.dim, c = e - g * p.dim;
-        reinterpret_cast<A*>(p.ck)[(((size_t)b * p.G + g) * p.slots + slot) * p.dim + c] = from_f<A>(ld_cg(row + p.off_k + e));
-    }
-    for (int e = threadIdx.x; e < p.G * p.vdim; e += blockDim.x) {
-        const int g = e / p.vdim, c = e - g * p.vdim;
-        reinterpret_cast<A*>(p.cv)[(((size_t)b * p.G + g) * p.slots + slot) * p.vdim + c] = from_f<A>(ld_cg(row + p.off_v + e));
-    }
+    const int g = blockIdx.z;
+    A* k = reinterpret_cast<A*>(p.ck) + (((size_t)b * p.G + g) * p.slots + slot) * p.dim;
+    A* v = reinterpret_cast<A*>(p.cv) + (((size_t)b * p.G + g) * p.slots + slot) * p.vdim;
+    for (int c = threadIdx.x; c < p.dim; c += blockDim.x) k[c] = from_f<A>(ld_cg(row + p.off_k + g * p.dim + c));
+    for (int c = threadIdx.x; c < p.vdim; c += blockDim.x) v[c] = from_f<A>(ld_cg(row + p.off_v + g * p.vdim + c));
 }
 
 // ------------------------------------------------------------------------------------------ one token
