@@ -7,11 +7,11 @@
 // with w = exp(-exp(-1/2) sigmoid(zw + w0)) and a = sigmoid(za + a_b); everything but the projections in fp32.
 //
 // Columns of S are independent of one another given the per-token vectors, so the prompt kernel gives each
-// CTA 16 columns of one head: four warps hold them in registers (lane = 8 row groups x 4 columns, packed
-// fp32 pairs) and walk the tokens, four more warps turn the projections of the NEXT 16 tokens into the fp32
-// vectors (u, w, a*u, k, r) in shared memory meanwhile.  A second kernel normalises and gates (the root mean
-// square runs over all columns of a head).  The decode kernel does one token of one head in one CTA, from the
-// projections to the gated output, the state read and written once.
+// CTA 32 columns of one head (16 beyond 128 key channels): a few warps hold them in registers and walk the tokens
+// four at a time, more warps turn the projections of the tokens ahead into the fp32 vectors they need, in shared
+// memory, meanwhile.  A second kernel normalises and gates (the root mean square runs over all columns of a head).
+// The decode kernel does one token of one head in one CTA, from the projections to the gated output, the state
+// read and written once.
 // A sequence starts with a zero state: position 0 ignores what the state buffer holds.
 #pragma once
 #include "decoder_common.cuh"
@@ -41,187 +41,322 @@ __device__ __forceinline__ float2 mul2(float2 a, float2 b) {
 }
 
 // ------------------------------------------------------------------------------------------ prompts
-constexpr int kScanCols = 16;
-template <int RPT>
+// Four tokens per step of the recurrence.  With S0 the state before them, p_j = u_j^T S_{j-1} (what the state
+// holds under key j), v'_j = |k_j| v_j and W_{i..j} the product of the decays of tokens i..j,
+//   p_j = c_j S0 + sum_{i<j} (A_ij v'_i - B_ij p_i)      c_j = W_{1..j-1} u_j    A_ij = u_j W_{i+1..j-1} u_i
+//   o_j = q_j S0 + sum_{i<=j} (C_ij v'_i - D_ij p_i)     q_j = W_{1..j} r_j      C_ij = r_j W_{i+1..j} u_i
+//   S4  = G S0 + sum_j (e_j v'_j - f_j p_j)              e_j = W_{j+1..4} u_j    f_j = a_j e_j    G = W_{1..4}
+// with B and D as A and C but a_i u_i in place of u_i.  Exact, no division, decay products of four factors at
+// most; one reduction over the key channels per four tokens on the critical path instead of four.  Places beyond
+// the prompt's end are filled with w = 1 and zeros, which leave the state as it is.
+//
+// What bounds it is the shared-memory pipe: a 16-byte load takes four of its cycles however many lanes read the
+// same address, so the cost of handing the vectors to the lanes is DK / (32 * CPT) cycles per vector and state
+// column - hence CPT = 4 columns per lane.
+constexpr int kScanTokens = 16;                             // tokens staged at a time: one block of four per producer warp
+template <int RL, int RPL, int CPT_>                        // consumer lanes over the key channels, state rows and columns per lane
 struct ScanShape {
-    static constexpr int DK = 8 * RPT;                      // padded key channels
-    static constexpr int CH = RPT > 16 ? 8 : 16;            // tokens staged at a time
-    static constexpr int TPW = CH / 4;                      // tokens per producer warp
+    static constexpr int DK = RL * RPL, CPT = CPT_;         // DK: padded key channels
     static constexpr int CPL = DK / 32;                     // channels per producer lane
-    static constexpr int smem = (2 * CH * 5 * DK + 2 * CH * kScanCols) * 4;
+    static constexpr int consumers = RL == 8 ? 2 : 4;       // consumer warps, 32 / RL * CPT state columns each
+    static constexpr int cols = 32 / RL * CPT * consumers;  // state columns per CTA
+    static constexpr int groups = CPL <= 2 ? 3 : 2;         // producer groups of four warps
+    static constexpr int threads = 32 * (consumers + 4 * groups);
+    static constexpr int sync = 32 * (consumers + 4);       // threads at a hand-over: the consumers and one group
+    static constexpr int val = 17 * DK;                     // a block: c, q, e, f of four tokens and G; then v' [4][cols];
+    static constexpr int sc = val + 4 * cols;               // then A, B [4][4] as [j][i], then C, D [4][4] as [j][i]
+    static constexpr int block = sc + 64;
+    static constexpr int buffers = CPL <= 2 ? 4 : CPL <= 4 ? 3 : 2;
+    static constexpr int smem = buffers * 4 * block * 4;
 };
 
-template <typename A, int RPT>
-__global__ void __launch_bounds__(256) delta_scan_kernel(const DeltaParams p) {
-    using L = ScanShape<RPT>;
-    constexpr int DK = L::DK, CH = L::CH;
-    extern __shared__ __align__(16) float scan_smem[];
-    float* vec = scan_smem;                                 // [2][CH][5][DK]: u, w, a*u, k, r
-    float* val = scan_smem + 2 * CH * 5 * DK;               // [2][CH][16]
+// hardware barriers 1 .. 15 between one side that waits and one that only arrives
+__device__ __forceinline__ void named_sync(int id, int threads) { asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(threads) : "memory"); }
+__device__ __forceinline__ void named_arrive(int id, int threads) { asm volatile("bar.arrive %0, %1;" ::"r"(id), "r"(threads) : "memory"); }
+
+template <typename A, int RL, int RPL, int CPT>
+__global__ void __launch_bounds__(ScanShape<RL, RPL, CPT>::threads) delta_scan_kernel(const DeltaParams p) {
+    using L = ScanShape<RL, RPL, CPT>;
+    constexpr int DK = L::DK, CH = kScanTokens, CPL = L::CPL, CW = L::consumers;
+    extern __shared__ __align__(16) float scan_smem[];      // [buffers][4 blocks][block]
     griddep_launch_dependents();
     griddep_wait();
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int c0 = blockIdx.x * kScanCols, head = blockIdx.y, b = blockIdx.z;
+    const int c0 = blockIdx.x * L::cols, head = blockIdx.y, b = blockIdx.z;
     const int T = p.T, dk = p.dk, dv = p.dv;
     const int chunks = (T + CH - 1) / CH;
     const size_t row0 = (size_t)b * T;
+    for (int i = tid; i < 4 * L::buffers * 64; i += L::threads) scan_smem[(i >> 6) * L::block + L::sc + (i & 63)] = 0.f;   // i > j stays zero
+    __syncthreads();
 
-    if (warp >= 4) {
-        // ------------------------------------------------ producers: projections -> fp32 vectors
-        const int pw = warp - 4;
+    // chunk c lies in buffer c mod buffers; producer group g makes the chunks c with c mod groups = g
+    const auto full = [](int c) { return 1 + c % L::buffers; };
+    const auto empty = [](int c) { return 1 + L::buffers + c % L::buffers; };
+    if (warp >= CW) {
+        // ------------------------------------------------ producers: projections -> vectors and scalars of a block
+        const int pw = warp & 3, group = (warp - CW) >> 2;
         const A* proj = reinterpret_cast<const A*>(p.proj);
-        float zk[L::TPW][L::CPL], zr[L::TPW][L::CPL], za[L::TPW][L::CPL], zw[L::TPW][L::CPL], zv[L::TPW];
-        float w0[L::CPL], ab[L::CPL];
+        // raw values of the next block: every address is clamped into the prompt and the loads are unconditional and
+        // unconverted, so that all of them are in flight at once; what lies outside is masked when they are used
+        Raw<A> rk[4][CPL], rr[4][CPL], ra[4][CPL], rv[4];
+        float rw[4][CPL];
+        float w0[CPL], ab[CPL];
 #pragma unroll
-        for (int j = 0; j < L::CPL; ++j) {
+        for (int j = 0; j < CPL; ++j) {
             const int c = lane + 32 * j;
             w0[j] = c < dk ? p.w0[head * dk + c] : 0.f;
             ab[j] = c < dk ? p.a_bias[head * dk + c] : 0.f;
         }
+        // where lane l's scalar goes: A and B (j > i) first, then C and D (j >= i)
+        int slot = 0;
+        {
+            int n = 0;
+            for (int m = 0; m < 2; ++m)
+                for (int j = 1; j < 4; ++j)
+                    for (int i = 0; i < j; ++i, ++n)
+                        if (n == lane) slot = m * 16 + j * 4 + i;
+            for (int m = 2; m < 4; ++m)
+                for (int j = 0; j < 4; ++j)
+                    for (int i = 0; i <= j; ++i, ++n)
+                        if (n == lane) slot = m * 16 + j * 4 + i;
+        }
         auto load = [&](int chunk) {
 #pragma unroll
-            for (int i = 0; i < L::TPW; ++i) {
-                const int t = chunk * CH + pw + 4 * i;
-                const bool live = t < T;
-                const A* row = proj + (row0 + (live ? t : 0)) * p.ld;
+            for (int i = 0; i < 4; ++i) {
+                const size_t r = row0 + min(chunk * CH + pw * 4 + i, T - 1);
+                const A* row = proj + r * p.ld;
 #pragma unroll
-                for (int j = 0; j < L::CPL; ++j) {
-                    const int c = lane + 32 * j;
-                    const bool ok = live && c < dk;
-                    zk[i][j] = ok ? ld_cg(row + p.off_k + head * dk + c) : 0.f;
-                    zr[i][j] = ok ? ld_cg(row + p.off_r + head * dk + c) : 0.f;
-                    za[i][j] = ok ? ld_cg(row + p.off_a + head * dk + c) : 0.f;
-                    zw[i][j] = ok ? ld_cg(p.zw + (row0 + t) * ((size_t)p.H * dk) + head * dk + c) : 0.f;
+                for (int j = 0; j < CPL; ++j) {
+                    const int c = head * dk + min(lane + 32 * j, dk - 1);
+                    rk[i][j].load(row + p.off_k + c);
+                    rr[i][j].load(row + p.off_r + c);
+                    ra[i][j].load(row + p.off_a + c);
+                    rw[i][j] = __ldcg(p.zw + r * ((size_t)p.H * dk) + c);
                 }
-                zv[i] = (live && lane < kScanCols && c0 + lane < dv) ? ld_cg(row + p.off_v + head * dv + c0 + lane) : 0.f;
+                rv[i].load(row + p.off_v + head * dv + min(c0 + (lane & (L::cols - 1)), dv - 1));
             }
         };
         auto emit = [&](int chunk) {
-            float* vb = vec + (size_t)(chunk & 1) * CH * 5 * DK;
-            float* wb = val + (chunk & 1) * CH * kScanCols;
+            float* blk = scan_smem + (size_t)(chunk % L::buffers * 4 + pw) * L::block;
+            float len[4], acc[32];
+            bool live[4];
 #pragma unroll
-            for (int i = 0; i < L::TPW; ++i) {
-                const int tt = pw + 4 * i;
-                float ss = 0.f;
+            for (int i = 0; i < 4; ++i) {
+                live[i] = chunk * CH + pw * 4 + i < T;
+                len[i] = 0.f;
 #pragma unroll
-                for (int j = 0; j < L::CPL; ++j) ss = fmaf(zk[i][j], zk[i][j], ss);
-                const float inv = 1.f / sqrtf(warp_sum(ss) + 1e-6f);
-#pragma unroll
-                for (int j = 0; j < L::CPL; ++j) {
-                    const int c = lane + 32 * j;
-                    const float u = zk[i][j] * inv;
-                    float* dst = vb + tt * 5 * DK + c;
-                    dst[0] = u;
-                    dst[DK] = __expf(-kDecayScale * sigmoid_f(zw[i][j] + w0[j]));
-                    dst[2 * DK] = sigmoid_f(za[i][j] + ab[j]) * u;
-                    dst[3 * DK] = zk[i][j];
-                    dst[4 * DK] = zr[i][j];
+                for (int j = 0; j < CPL; ++j) {
+                    const float k = live[i] && lane + 32 * j < dk ? rk[i][j].get() : 0.f;
+                    len[i] = fmaf(k, k, len[i]);
                 }
-                if (lane < kScanCols) wb[tt * kScanCols + lane] = zv[i];
             }
+#pragma unroll
+            for (int d = 16; d; d >>= 1)
+#pragma unroll
+                for (int i = 0; i < 4; ++i) len[i] += __shfl_xor_sync(0xffffffffu, len[i], d);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                len[i] = sqrtf(len[i] + 1e-6f);
+                if (lane < L::cols) blk[L::val + i * L::cols + lane] = live[i] && c0 + lane < dv ? rv[i].get() * len[i] : 0.f;
+                len[i] = 1.f / len[i];
+            }
+#pragma unroll
+            for (int n = 0; n < 32; ++n) acc[n] = 0.f;
+#pragma unroll
+            for (int j = 0; j < CPL; ++j) {
+                const int c = lane + 32 * j;
+                float w[4], u[4], a[4], r[4], au[4];
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    const bool in = live[i] && c < dk;
+                    u[i] = in ? rk[i][j].get() * len[i] : 0.f;
+                    w[i] = in ? __expf(-kDecayScale * sigmoid_fast(rw[i][j] + w0[j])) : 1.f;
+                    a[i] = sigmoid_fast(ra[i][j].get() + ab[j]);
+                    r[i] = in ? rr[i][j].get() : 0.f;
+                    au[i] = a[i] * u[i];
+                }
+                const float w01 = w[0] * w[1], w23 = w[2] * w[3], w12 = w[1] * w[2];
+                const float w012 = w01 * w[2], w123 = w[1] * w23, w0123 = w01 * w23;
+                float* d = blk + c;
+                d[0 * DK] = u[0], d[1 * DK] = w[0] * u[1], d[2 * DK] = w01 * u[2], d[3 * DK] = w012 * u[3];               // c
+                d[4 * DK] = w[0] * r[0], d[5 * DK] = w01 * r[1], d[6 * DK] = w012 * r[2], d[7 * DK] = w0123 * r[3];      // q
+                const float e0 = w123 * u[0], e1 = w23 * u[1], e2 = w[3] * u[2], e3 = u[3];
+                d[8 * DK] = e0, d[9 * DK] = e1, d[10 * DK] = e2, d[11 * DK] = e3;
+                d[12 * DK] = a[0] * e0, d[13 * DK] = a[1] * e1, d[14 * DK] = a[2] * e2, d[15 * DK] = a[3] * e3;          // f
+                d[16 * DK] = w0123;
+                const float x[6] = {u[1], u[2] * w[1], u[2], u[3] * w12, u[3] * w[2], u[3]};                             // (1,0) (2,0) (2,1) (3,0) (3,1) (3,2)
+                const float y[10] = {r[0], r[1] * w[1], r[1], r[2] * w12, r[2] * w[2], r[2], r[3] * w123, r[3] * w23, r[3] * w[3], r[3]};
+                int n = 0;
+#pragma unroll
+                for (int t = 1; t < 4; ++t)
+#pragma unroll
+                    for (int i = 0; i < t; ++i, ++n) acc[n] = fmaf(x[n], u[i], acc[n]), acc[6 + n] = fmaf(x[n], au[i], acc[6 + n]);
+                n = 0;
+#pragma unroll
+                for (int t = 0; t < 4; ++t)
+#pragma unroll
+                    for (int i = 0; i <= t; ++i, ++n) acc[12 + n] = fmaf(y[n], u[i], acc[12 + n]), acc[22 + n] = fmaf(y[n], au[i], acc[22 + n]);
+            }
+            if (chunk + L::groups < chunks) load(chunk + L::groups);   // underneath the sums
+            // 32 sums over 32 lanes: a transposing butterfly leaves sum l in lane l
+#pragma unroll
+            for (int d = 16; d; d >>= 1)
+#pragma unroll
+                for (int i = 0; i < d; ++i) {
+                    const float keep = (lane & d) ? acc[i + d] : acc[i], give = (lane & d) ? acc[i] : acc[i + d];
+                    acc[i] = keep + __shfl_xor_sync(0xffffffffu, give, d);
+                }
+            blk[L::sc + slot] = acc[0];
         };
-        load(0);
-        emit(0);
-        if (chunks > 1) load(1);
-        __syncthreads();
-        for (int c = 0; c < chunks; ++c) {
-            if (c + 1 < chunks) {
-                emit(c + 1);
-                if (c + 2 < chunks) load(c + 2);
-            }
-            __syncthreads();
+        if (group < chunks) load(group);
+        for (int c = group; c < chunks; c += L::groups) {
+            if (c >= L::buffers) named_sync(empty(c), L::sync);
+            emit(c);
+            named_arrive(full(c), L::sync);
         }
         return;
     }
 
-    // -------------------------------------------------- consumers: the recurrence
-    const int ks = lane & 7, cl = warp * 4 + (lane >> 3), col = c0 + cl;
-    const bool live_col = col < dv;
-    float2 s[RPT / 2];                                      // rows 32*i + 4*ks + 0..3, i = 0 .. RPT/4 - 1
+    // -------------------------------------------------- consumers: lane = RL row groups x 32 / RL groups of CPT columns
+    constexpr int PAIRS = RPL / 2, REM = 8 * CPT / RL;      // REM: sums left per lane of the 8 * CPT products
+    const int ks = lane & (RL - 1), cl = warp * (32 / RL * CPT) + lane / RL * CPT, col = c0 + cl;
+    float2 s[CPT][PAIRS];                                   // rows 4*RL*i + 4*ks + 0 .. 3
     float* st = p.state + ((size_t)b * p.H + head) * dk * dv;
     const bool fresh = p.pos[0] == 0;
+    auto row_of = [&](int pair, int e) { return (pair >> 1) * (4 * RL) + 4 * ks + 2 * (pair & 1) + e; };
 #pragma unroll
-    for (int i = 0; i < RPT / 4; ++i) {
-        float f[4];
+    for (int x = 0; x < CPT; ++x)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            const int k = 32 * i + 4 * ks + e;
-            f[e] = (!fresh && live_col && k < dk) ? ld_cg(st + (size_t)k * dv + col) : 0.f;
+        for (int i = 0; i < PAIRS; ++i) {
+            float f[2];
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const int k = row_of(i, e);
+                f[e] = (!fresh && col + x < dv && k < dk) ? ld_cg(st + (size_t)k * dv + col + x) : 0.f;
+            }
+            s[x][i] = make_float2(f[0], f[1]);
         }
-        s[2 * i] = make_float2(f[0], f[1]), s[2 * i + 1] = make_float2(f[2], f[3]);
-    }
-    __syncthreads();
+    auto vec = [&](const float* src, float2 (&v)[PAIRS]) {
+#pragma unroll
+        for (int i = 0; i < RPL / 4; ++i) {
+            const float4 q = *reinterpret_cast<const float4*>(src + 4 * RL * i + 4 * ks);
+            v[2 * i] = make_float2(q.x, q.y), v[2 * i + 1] = make_float2(q.z, q.w);
+        }
+    };
+    const int n0 = ks * REM, jo = (n0 / CPT) & 3, x0 = n0 % CPT;   // the sums of this lane: product n0 / CPT, columns x0 ..
     for (int c = 0; c < chunks; ++c) {
-        const float* vb = vec + (size_t)(c & 1) * CH * 5 * DK + 4 * ks;
-        const float* wb = val + (c & 1) * CH * kScanCols + cl;
-        const int n = min(CH, T - c * CH);
-        for (int t8 = 0; t8 < n; t8 += 8) {
-            float part[8];
+        const int blocks = min(4, (T - c * CH + 3) >> 2);
+        named_sync(full(c), L::sync);
+#pragma unroll 1
+        for (int q = 0; q < blocks; ++q) {
+            const float* blk = scan_smem + (size_t)(c % L::buffers * 4 + q) * L::block;
+            // products with the state before the block: c_j, then q_j, column x in place (4 * kind + j) * CPT + x
+            float d[8 * CPT];
+            float2 v[PAIRS];
 #pragma unroll
             for (int j = 0; j < 8; ++j) {
-                part[j] = 0.f;
-                if (t8 + j < n) {
-                    const float* q = vb + (t8 + j) * 5 * DK;
-                    float2 d0 = make_float2(0.f, 0.f), d1 = d0;
+                vec(blk + j * DK, v);
 #pragma unroll
-                    for (int i = 0; i < RPT / 4; ++i) {
-                        const float4 u = *reinterpret_cast<const float4*>(q + 32 * i);
-                        d0 = fma2(make_float2(u.x, u.y), s[2 * i], d0);
-                        d1 = fma2(make_float2(u.z, u.w), s[2 * i + 1], d1);
-                    }
-                    float seen = (d0.x + d0.y) + (d1.x + d1.y);
-                    seen += __shfl_xor_sync(0xffffffffu, seen, 1);
-                    seen += __shfl_xor_sync(0xffffffffu, seen, 2);
-                    seen += __shfl_xor_sync(0xffffffffu, seen, 4);
-                    const float2 neg = make_float2(-seen, -seen);
-                    const float v = wb[(t8 + j) * kScanCols];
-                    const float2 vv = make_float2(v, v);
-                    float2 o0 = make_float2(0.f, 0.f), o1 = o0;
+                for (int x = 0; x < CPT; ++x) {
+                    float2 t = mul2(v[0], s[x][0]);
 #pragma unroll
-                    for (int i = 0; i < RPT / 4; ++i) {
-                        const float4 w = *reinterpret_cast<const float4*>(q + DK + 32 * i);
-                        const float4 au = *reinterpret_cast<const float4*>(q + 2 * DK + 32 * i);
-                        const float4 k = *reinterpret_cast<const float4*>(q + 3 * DK + 32 * i);
-                        const float4 r = *reinterpret_cast<const float4*>(q + 4 * DK + 32 * i);
-                        // decayed state plus the new pair does not wait for the removal term
-                        const float2 m0 = fma2(make_float2(w.x, w.y), s[2 * i], mul2(make_float2(k.x, k.y), vv));
-                        const float2 m1 = fma2(make_float2(w.z, w.w), s[2 * i + 1], mul2(make_float2(k.z, k.w), vv));
-                        s[2 * i] = fma2(make_float2(au.x, au.y), neg, m0);
-                        s[2 * i + 1] = fma2(make_float2(au.z, au.w), neg, m1);
-                        o0 = fma2(make_float2(r.x, r.y), s[2 * i], o0);
-                        o1 = fma2(make_float2(r.z, r.w), s[2 * i + 1], o1);
-                    }
-                    part[j] = (o0.x + o0.y) + (o1.x + o1.y);
+                    for (int i = 1; i < PAIRS; ++i) t = fma2(v[i], s[x][i], t);
+                    d[j * CPT + x] = t.x + t.y;
                 }
             }
-            // eight partial outputs over eight row groups: a transposing butterfly leaves token t8 + ks in lane ks
-            float h4[4], h2[2];
+#pragma unroll
+            for (int h = RL / 2; h; h >>= 1)
+#pragma unroll
+                for (int i = 0; i < h * REM; ++i) {
+                    const float keep = (ks & h) ? d[i + h * REM] : d[i], give = (ks & h) ? d[i] : d[i + h * REM];
+                    d[i] = keep + __shfl_xor_sync(0xffffffffu, give, h);
+                }
+            float val[4][CPT], pj[4][CPT];
+            vec(blk + 16 * DK, v);
+#pragma unroll
+            for (int x = 0; x < CPT; ++x)
+#pragma unroll
+                for (int i = 0; i < PAIRS; ++i) s[x][i] = mul2(v[i], s[x][i]);
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
-                const float keep = (ks & 4) ? part[j + 4] : part[j], give = (ks & 4) ? part[j] : part[j + 4];
-                h4[j] = keep + __shfl_xor_sync(0xffffffffu, give, 4);
+                const float* src = blk + L::val + j * L::cols + cl;
+                if constexpr (CPT == 4) {
+                    const float4 t = *reinterpret_cast<const float4*>(src);
+                    val[j][0] = t.x, val[j][1] = t.y, val[j][2] = t.z, val[j][3] = t.w;
+                } else {
+                    const float2 t = *reinterpret_cast<const float2*>(src);
+                    val[j][0] = t.x, val[j][1] = t.y;
+                }
+                vec(blk + (8 + j) * DK, v);
+#pragma unroll
+                for (int x = 0; x < CPT; ++x)
+#pragma unroll
+                    for (int i = 0; i < PAIRS; ++i) s[x][i] = fma2(v[i], make_float2(val[j][x], val[j][x]), s[x][i]);
+            }
+            const float* sc = blk + L::sc;
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+#pragma unroll
+                for (int x = 0; x < CPT; ++x) {
+                    const int n = j * CPT + x;
+                    pj[j][x] = __shfl_sync(0xffffffffu, d[n % REM], (lane & ~(RL - 1)) | (n / REM));
+                }
+            // what does not depend on p first, then the triangular solve
+            float bj[4][3];
+#pragma unroll
+            for (int j = 1; j < 4; ++j) {
+                const float4 a = *reinterpret_cast<const float4*>(sc + 4 * j), bb = *reinterpret_cast<const float4*>(sc + 16 + 4 * j);
+                const float aj[3] = {a.x, a.y, a.z};
+                bj[j][0] = bb.x, bj[j][1] = bb.y, bj[j][2] = bb.z;
+#pragma unroll
+                for (int x = 0; x < CPT; ++x)
+#pragma unroll
+                    for (int i = 0; i < j; ++i) pj[j][x] = fmaf(aj[i], val[i][x], pj[j][x]);
             }
 #pragma unroll
-            for (int j = 0; j < 2; ++j) {
-                const float keep = (ks & 2) ? h4[j + 2] : h4[j], give = (ks & 2) ? h4[j] : h4[j + 2];
-                h2[j] = keep + __shfl_xor_sync(0xffffffffu, give, 2);
+            for (int i = 0; i < 3; ++i)
+#pragma unroll
+                for (int j = i + 1; j < 4; ++j)
+#pragma unroll
+                    for (int x = 0; x < CPT; ++x) pj[j][x] = fmaf(-bj[j][i], pj[i][x], pj[j][x]);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                vec(blk + (12 + j) * DK, v);
+#pragma unroll
+                for (int x = 0; x < CPT; ++x)
+#pragma unroll
+                    for (int i = 0; i < PAIRS; ++i) s[x][i] = fma2(v[i], make_float2(-pj[j][x], -pj[j][x]), s[x][i]);
             }
-            const float keep = (ks & 1) ? h2[1] : h2[0], give = (ks & 1) ? h2[0] : h2[1];
-            const float o = keep + __shfl_xor_sync(0xffffffffu, give, 1);
-            const int t = c * CH + t8 + ks;
-            if (t8 + ks < n && live_col) p.o[(row0 + t) * ((size_t)p.H * dv) + (size_t)head * dv + col] = o;
+            // the upper half of the lanes holds q_j S0: the outputs of token jo
+            const int t = c * CH + 4 * q + jo;
+            const float4 cc = *reinterpret_cast<const float4*>(sc + 32 + 4 * jo), dd = *reinterpret_cast<const float4*>(sc + 48 + 4 * jo);
+            float* out = p.o + (row0 + t) * ((size_t)p.H * dv) + (size_t)head * dv + col + x0;
+#pragma unroll
+            for (int i = 0; i < REM; ++i) {
+                float vx[4], px[4];                          // column x0 + i
+#pragma unroll
+                for (int m = 0; m < 4; ++m) {
+                    vx[m] = val[m][i], px[m] = pj[m][i];
+#pragma unroll
+                    for (int x = REM; x < CPT; x += REM)
+                        if (x0 == x) vx[m] = val[m][x + i], px[m] = pj[m][x + i];
+                }
+                const float o = fmaf(cc.x, vx[0], fmaf(cc.y, vx[1], fmaf(cc.z, vx[2], fmaf(cc.w, vx[3], d[i]))));
+                const float o2 = fmaf(dd.x, px[0], fmaf(dd.y, px[1], fmaf(dd.z, px[2], dd.w * px[3])));
+                if (ks >= RL / 2 && t < T && col + x0 + i < dv) out[i] = o - o2;
+            }
         }
-        __syncthreads();
+        if (c + L::buffers < chunks) named_arrive(empty(c), L::sync);
     }
 #pragma unroll
-    for (int i = 0; i < RPT / 4; ++i) {
-        const float f[4] = {s[2 * i].x, s[2 * i].y, s[2 * i + 1].x, s[2 * i + 1].y};
+    for (int x = 0; x < CPT; ++x)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            const int k = 32 * i + 4 * ks + e;
-            if (live_col && k < dk) st[(size_t)k * dv + col] = f[e];
-        }
-    }
+        for (int i = 0; i < PAIRS; ++i)
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const int k = row_of(i, e);
+                if (col + x < dv && k < dk) st[(size_t)k * dv + col + x] = e ? s[x][i].y : s[x][i].x;
+            }
 }
 
 // y = o / rms(o) * norm * sigmoid(gate), one warp per row and head
