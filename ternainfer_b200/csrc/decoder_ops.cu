@@ -90,19 +90,19 @@ static int hyper(const HyperParams& p, int pdl, void* stream) {
 
 static bool quads(int n) { return n >= 4 && n <= 128 && (n & (n - 1)) == 0; }
 
-template <typename A, int RL, int RPL, int CPT>
+template <typename A, int RL, int RPL, int CPT, int CW, int GR>
 static int delta_scan(const DeltaParams& p, int pdl, void* stream) {
-    using L = ScanShape<RL, RPL, CPT>;
-    return launch(delta_scan_kernel<A, RL, RPL, CPT>, dim3((p.dv + L::cols - 1) / L::cols, p.H, p.B), L::threads, L::smem, pdl, stream, 1, p);
+    using L = ScanShape<RL, RPL, CPT, CW, GR>;
+    return launch(delta_scan_kernel<A, RL, RPL, CPT, CW, GR>, dim3((p.dv + L::cols - 1) / L::cols, p.H, p.B), L::threads, L::smem, pdl, stream, 1, p);
 }
 
 template <typename A>
 static int delta_prompt(const DeltaParams& p, int pdl, void* stream) {
     int rc;
-    if (p.dk <= 32) rc = delta_scan<A, 8, 4, 4>(p, pdl, stream);
-    else if (p.dk <= 64) rc = delta_scan<A, 16, 4, 4>(p, pdl, stream);
-    else if (p.dk <= 128) rc = delta_scan<A, 16, 8, 4>(p, pdl, stream);
-    else rc = delta_scan<A, 16, 16, 2>(p, pdl, stream);
+    if (p.dk <= 32) rc = delta_scan<A, 8, 4, 4, 2, 2>(p, pdl, stream);
+    else if (p.dk <= 64) rc = delta_scan<A, 16, 4, 2, 8, 2>(p, pdl, stream);
+    else if (p.dk <= 128) rc = delta_scan<A, 16, 8, 4, 4, 2>(p, pdl, stream);
+    else rc = delta_scan<A, 16, 16, 2, 4, 2>(p, pdl, stream);
     if (rc) return rc;
     const long long units = (long long)p.B * p.T * p.H;
     if (quads(p.dv) && p.ld % 4 == 0 && p.off_g % 4 == 0 && !misaligned(p.proj, 16) && !misaligned(p.y, 16) && !misaligned(p.norm, 16))

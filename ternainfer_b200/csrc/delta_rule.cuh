@@ -50,17 +50,19 @@ __device__ __forceinline__ float2 mul2(float2 a, float2 b) {
 // most; one reduction over the key channels per four tokens on the critical path instead of four.  Places beyond
 // the prompt's end are filled with w = 1 and zeros, which leave the state as it is.
 //
-// What bounds it is the shared-memory pipe: a 16-byte load takes four of its cycles however many lanes read the
-// same address, so the cost of handing the vectors to the lanes is DK / (32 * CPT) cycles per vector and state
-// column - hence CPT = 4 columns per lane.
+// Two costs pull against each other.  A 16-byte shared load takes four cycles of its pipe however many lanes read
+// the same address, so handing the vectors to the lanes costs DK / (32 * CPT) cycles per vector and state column:
+// few columns per lane fill that pipe.  Many columns per lane make a warp's chain of dependent instructions per
+// four tokens longer, and that chain is what the recurrence waits for.  The shapes chosen by the host were measured.
 constexpr int kScanTokens = 16;                             // tokens staged at a time: one block of four per producer warp
-template <int RL, int RPL, int CPT_>                        // consumer lanes over the key channels, state rows and columns per lane
+// RL consumer lanes over the key channels, RPL state rows and CPT columns per lane, CW consumer warps, GR producer groups
+template <int RL, int RPL, int CPT_, int CW, int GR>
 struct ScanShape {
     static constexpr int DK = RL * RPL, CPT = CPT_;         // DK: padded key channels
     static constexpr int CPL = DK / 32;                     // channels per producer lane
-    static constexpr int consumers = RL == 8 ? 2 : 4;       // consumer warps, 32 / RL * CPT state columns each
+    static constexpr int consumers = CW;                    // 32 / RL * CPT state columns each
     static constexpr int cols = 32 / RL * CPT * consumers;  // state columns per CTA
-    static constexpr int groups = CPL <= 2 ? 3 : 2;         // producer groups of four warps
+    static constexpr int groups = GR;                       // of four producer warps
     static constexpr int threads = 32 * (consumers + 4 * groups);
     static constexpr int sync = 32 * (consumers + 4);       // threads at a hand-over: the consumers and one group
     static constexpr int val = 17 * DK;                     // a block: c, q, e, f of four tokens and G; then v' [4][cols];
@@ -74,10 +76,10 @@ struct ScanShape {
 __device__ __forceinline__ void named_sync(int id, int threads) { asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(threads) : "memory"); }
 __device__ __forceinline__ void named_arrive(int id, int threads) { asm volatile("bar.arrive %0, %1;" ::"r"(id), "r"(threads) : "memory"); }
 
-template <typename A, int RL, int RPL, int CPT>
-__global__ void __launch_bounds__(ScanShape<RL, RPL, CPT>::threads) delta_scan_kernel(const DeltaParams p) {
-    using L = ScanShape<RL, RPL, CPT>;
-    constexpr int DK = L::DK, CH = kScanTokens, CPL = L::CPL, CW = L::consumers;
+template <typename A, int RL, int RPL, int CPT, int CW, int GR>
+__global__ void __launch_bounds__(ScanShape<RL, RPL, CPT, CW, GR>::threads) delta_scan_kernel(const DeltaParams p) {
+    using L = ScanShape<RL, RPL, CPT, CW, GR>;
+    constexpr int DK = L::DK, CH = kScanTokens, CPL = L::CPL;
     extern __shared__ __align__(16) float scan_smem[];      // [buffers][4 blocks][block]
     griddep_launch_dependents();
     griddep_wait();
@@ -94,7 +96,7 @@ __global__ void __launch_bounds__(ScanShape<RL, RPL, CPT>::threads) delta_scan_k
     const auto empty = [](int c) { return 1 + L::buffers + c % L::buffers; };
     if (warp >= CW) {
         // ------------------------------------------------ producers: projections -> vectors and scalars of a block
-        const int pw = warp & 3, group = (warp - CW) >> 2;
+        const int pw = (warp - CW) & 3, group = (warp - CW) >> 2;
         const A* proj = reinterpret_cast<const A*>(p.proj);
         // raw values of the next block: every address is clamped into the prompt and the loads are unconditional and
         // unconverted, so that all of them are in flight at once; what lies outside is masked when they are used
@@ -133,7 +135,7 @@ __global__ void __launch_bounds__(ScanShape<RL, RPL, CPT>::threads) delta_scan_k
                     ra[i][j].load(row + p.off_a + c);
                     rw[i][j] = __ldcg(p.zw + r * ((size_t)p.H * dk) + c);
                 }
-                rv[i].load(row + p.off_v + head * dv + min(c0 + (lane & (L::cols - 1)), dv - 1));
+                rv[i].load(row + p.off_v + head * dv + min(c0 + min(lane, L::cols - 1), dv - 1));
             }
         };
         auto emit = [&](int chunk) {
@@ -157,6 +159,7 @@ __global__ void __launch_bounds__(ScanShape<RL, RPL, CPT>::threads) delta_scan_k
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
                 len[i] = sqrtf(len[i] + 1e-6f);
+                static_assert(L::cols <= 32, "one producer lane per column");
                 if (lane < L::cols) blk[L::val + i * L::cols + lane] = live[i] && c0 + lane < dv ? rv[i].get() * len[i] : 0.f;
                 len[i] = 1.f / len[i];
             }

@@ -24,6 +24,13 @@ from .cache import CachePool, SequenceCache
 from .model import ModelArgs, Transformer
 
 
+def _check_status(model):
+    """Models whose kernels report failures on the device raise here."""
+    check = getattr(model, "check_status", None)
+    if check is not None:
+        check()
+
+
 @dataclass
 class GenArgs:
     gen_length: int = 128
@@ -90,6 +97,7 @@ class FastGen:
                 nxt = self.model(self._tokens, self.cache, self._pos, greedy_last=True)
         torch.cuda.synchronize()
         t2 = time.perf_counter()
+        _check_status(self.model)
         stats = {"prefill_s": t1 - t0, "decode_s": t2 - t1,
                  "prefill_tokens_per_s": a.gen_bsz * a.prompt_length / (t1 - t0),
                  "decode_tokens_per_s": a.gen_bsz * (a.gen_length - 1) / (t2 - t1)}
@@ -152,11 +160,18 @@ class StepEngine:
             if graph is None:
                 graph = self._graphs[id(r.cache)] = _StepGraph(self.model, r.cache, self.device)
             logits = graph.run(tokens[0], start)
-            return logits if want else None
+            if not want:
+                return None
+            logits = logits.clone()         # the next replay writes the same buffer
+            _check_status(self.model)
+            return logits
         logits = self.model(torch.tensor([tokens], device=self.device), r.cache,
                             torch.arange(start, r.length, device=self.device),
                             want=torch.tensor(want or [len(tokens) - 1], device=self.device))
-        return logits[0] if want else None
+        if not want:
+            return None
+        _check_status(self.model)
+        return logits[0]
 
     def finish(self, request: str):
         self.pool.release(self.live.pop(request).cache)

@@ -19,6 +19,7 @@ from torch import nn
 
 from . import decoder_ops as ops
 from .cache import SequenceCache
+from .lib import check, load_decoder_library
 from .mixers import GeneralDelta, SigmoidAttention, SquaredReluFeedForward, _param
 
 
@@ -199,6 +200,10 @@ class Kepovik(nn.Module):
         if greedy_last:
             return ops.output_argmax(h, self.head)
         return ops.output_logits(h, self.head).view(B, -1, a.vocab)
+
+    def check_status(self):
+        """Raise if a bounded wait inside a kernel has run out since the last call (synchronises)."""
+        check(load_decoder_library().decoder_status())
 
     @staticmethod
     def _after(x, write):
