@@ -2,8 +2,10 @@
 
 ``SequenceCache`` is what ``make_cache`` of every model returns and ``forward``
 of every model takes: a list with one entry per layer - a (keys, values) pair
-of an attention layer, the state tensor of a recurrent one - plus the last
-token of every sequence for models whose embedding looks back.  Nothing in it
+of an attention layer, one tensor of latents of an attention layer that shares
+them among its heads, the state of a recurrent one, nothing for a layer that
+reads another layer's entry - plus the last token of every sequence for models
+whose embedding looks back.  Nothing in it
 has to be cleared between sequences: attention reads only positions that the
 sequence has written, and the kernels of recurrent layers and of the token
 history start from nothing at position 0.
@@ -32,6 +34,11 @@ def chunk_kv_cache(batch: int, kv_heads: int, slots: int, dim: int, vdim: int, d
     start of a chunk of ``slots`` positions: position p lives in slot p mod chunk."""
     return (torch.zeros((batch, kv_heads, slots, dim), device=device, dtype=dtype),
             torch.zeros((batch, kv_heads, slots, vdim), device=device, dtype=dtype))
+
+
+def latent_cache(batch: int, slots: int, ld: int, device, dtype):
+    """Latents and shared key parts [B, slots, ld] of an attention layer: position p lives in slot p."""
+    return torch.zeros((batch, slots, ld), device=device, dtype=dtype)
 
 
 class CachePool:

@@ -24,22 +24,6 @@ constexpr float kDecayScale = 0.60653065971263342f;   // exp(-1/2)
 
 typedef decoder_delta_args DeltaParams;
 
-__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
-    float2 d;
-    asm("fma.rn.f32x2 %0, %1, %2, %3;"
-        : "=l"(reinterpret_cast<unsigned long long&>(d))
-        : "l"(reinterpret_cast<const unsigned long long&>(a)), "l"(reinterpret_cast<const unsigned long long&>(b)),
-          "l"(reinterpret_cast<const unsigned long long&>(c)));
-    return d;
-}
-__device__ __forceinline__ float2 mul2(float2 a, float2 b) {
-    float2 d;
-    asm("mul.rn.f32x2 %0, %1, %2;"
-        : "=l"(reinterpret_cast<unsigned long long&>(d))
-        : "l"(reinterpret_cast<const unsigned long long&>(a)), "l"(reinterpret_cast<const unsigned long long&>(b)));
-    return d;
-}
-
 // ------------------------------------------------------------------------------------------ prompts
 // Four tokens per step of the recurrence.  With S0 the state before them, p_j = u_j^T S_{j-1} (what the state
 // holds under key j), v'_j = |k_j| v_j and W_{i..j} the product of the decays of tokens i..j,
@@ -413,17 +397,6 @@ __global__ void __launch_bounds__(256) delta_finish4_kernel(const DeltaParams p)
         if (at[i] < total)
             st4(reinterpret_cast<A*>(p.y) + at[i], make_float4(o[i].x * inv * w.x * sigmoid_fast(g[i].x), o[i].y * inv * w.y * sigmoid_fast(g[i].y),
                                                                o[i].z * inv * w.z * sigmoid_fast(g[i].z), o[i].w * inv * w.w * sigmoid_fast(g[i].w)));
-    }
-}
-
-// t1[row][j] = tanh of the low-rank decay projection, contiguous (input of the second projection of a prompt)
-template <typename A>
-__global__ void __launch_bounds__(256) tanh_cols_kernel(const A* proj, long long ld, int off, int rank, long long rows, A* out) {
-    griddep_launch_dependents();
-    griddep_wait();
-    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < rows * rank; i += (long long)gridDim.x * blockDim.x) {
-        const long long r = i / rank;
-        out[i] = from_f<A>(tanhf(ld_cg(proj + r * ld + off + (i - r * rank))));
     }
 }
 

@@ -3,10 +3,14 @@
 //
 // The streams live in fp32, x [rows][S][D].  One launch does what stands between two sublayers:
 //   x_t <- sum_s mix[s][t] x_s + m * out[t] * y        (write the previous sublayer's output y back)
+// where, for a single stream, y may be the sum of two sublayers' outputs, the second optionally a weighted sum of gathered rows (the
+// chosen experts of a token); without mix and out the streams stay apart and y goes to all of them.
 //   u = sum_s in[s] x_s                                (read for the next one)
 //   h = u / sqrt(mean(u^2) + eps) * (w_offset + w)     (its norm, rounded to the activation type)
 // Without y it only reads (first sublayer); with in = null the read is the plain sum of the streams
 // (final norm); with a row list it reads and normalises those rows only and leaves x alone.
+// In a decode step of a single stream the same launch makes the inputs of projections that look one token back:
+//   mixed_j = h + (h_before - h) * mu_j                 (h_before: the sequence's previous h, kept in prev)
 // One CTA per row; HBM traffic: the streams once in, once out, y in, h out.
 #pragma once
 #include "decoder_common.cuh"
@@ -48,6 +52,12 @@ __global__ void __launch_bounds__(256) embed_kernel(const EmbedParams p) {
 
 typedef decoder_hyper_args HyperParams;
 
+__device__ __forceinline__ float shifted(float h, float before, float mu) { return fmaf(before - h, mu, h); }
+template <typename A>
+__device__ __forceinline__ float4 round_to(float4 v) {
+    return make_float4(to_f(from_f<A>(v.x)), to_f(from_f<A>(v.y)), to_f(from_f<A>(v.z)), to_f(from_f<A>(v.w)));
+}
+
 template <typename A, int S, int V>
 __global__ void __launch_bounds__(1024) hyper_kernel(const HyperParams p) {
     extern __shared__ __align__(16) float u_s[];
@@ -56,8 +66,8 @@ __global__ void __launch_bounds__(1024) hyper_kernel(const HyperParams p) {
     griddep_launch_dependents();
     const int tid = threadIdx.x, D = p.D;
     for (int i = tid; i < S * S + 2 * S; i += blockDim.x) {
-        if (i < S * S) coef[i] = p.y ? p.mix[i] : 0.f;
-        else if (i < S * S + S) coef[i] = p.y ? p.m * p.out[i - S * S] : 0.f;
+        if (i < S * S) coef[i] = p.mix ? p.mix[i] : i % (S + 1) == 0 ? 1.f : 0.f;
+        else if (i < S * S + S) coef[i] = p.out ? p.m * p.out[i - S * S] : p.m;
         else coef[i] = p.in ? p.in[i - S * S - S] : 1.f;
     }
     __syncthreads();
@@ -73,6 +83,9 @@ __global__ void __launch_bounds__(1024) hyper_kernel(const HyperParams p) {
     const size_t row = p.rows ? (size_t)p.rows[blockIdx.x] : (size_t)blockIdx.x;
     float* xr = p.x + row * S * D;
     const A* yr = reinterpret_cast<const A*>(p.y) + row * D;
+    const A* y2 = reinterpret_cast<const A*>(p.y2);
+    const int n2 = S == 1 && p.y2 ? (p.top > 0 ? p.top : 1) : 0;
+    const int n_mu = S == 1 ? p.n_mu : 0;
     const bool store = p.y && !p.rows;
     float ss = 0.f;
     for (int d = tid * V; d < D; d += blockDim.x * V) {
@@ -93,6 +106,16 @@ __global__ void __launch_bounds__(1024) hyper_kernel(const HyperParams p) {
                 y[0] = v.x, y[1] = v.y, y[2] = v.z, y[3] = v.w;
             } else {
                 y[0] = ld_cg(yr + d);
+            }
+            for (int j = 0; j < n2; ++j) {
+                const size_t r2 = p.top > 0 ? (size_t)__ldcg(p.slots + row * p.top + j) : row;
+                const float w2 = p.top > 0 ? __ldcg(p.slot_w + row * p.top + j) : 1.f;
+                if constexpr (V == 4) {
+                    const float4 v = ld_cg4(y2 + r2 * D + d);
+                    y[0] = fmaf(w2, v.x, y[0]), y[1] = fmaf(w2, v.y, y[1]), y[2] = fmaf(w2, v.z, y[2]), y[3] = fmaf(w2, v.w, y[3]);
+                } else {
+                    y[0] = fmaf(w2, ld_cg(y2 + r2 * D + d), y[0]);
+                }
             }
 #pragma unroll
             for (int t = 0; t < S; ++t)
@@ -125,33 +148,70 @@ __global__ void __launch_bounds__(1024) hyper_kernel(const HyperParams p) {
     if (!p.h) return;
     const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)D + p.eps);
     A* h = reinterpret_cast<A*>(p.h) + (size_t)blockIdx.x * D;
+    const bool first = n_mu > 0 && p.pos[0] == 0;
+    A* prev = reinterpret_cast<A*>(p.prev) + row * D;
+    A* mixed = reinterpret_cast<A*>(p.mixed) + (size_t)blockIdx.x * D;
     for (int d = tid * V; d < D; d += blockDim.x * V) {   // each thread reads back what it wrote itself
         if constexpr (V == 4) {
             const float4 w = *reinterpret_cast<const float4*>(p.w + d);
             const float4 u = *reinterpret_cast<const float4*>(u_s + d);
-            st4(h + d, make_float4(u.x * inv * (p.w_offset + w.x), u.y * inv * (p.w_offset + w.y),
-                                   u.z * inv * (p.w_offset + w.z), u.w * inv * (p.w_offset + w.w)));
+            float4 n = make_float4(u.x * inv * (p.w_offset + w.x), u.y * inv * (p.w_offset + w.y), u.z * inv * (p.w_offset + w.z),
+                                   u.w * inv * (p.w_offset + w.w));
+            st4(h + d, n);
+            if (n_mu > 0) {
+                const float4 b = first ? make_float4(0.f, 0.f, 0.f, 0.f) : ld_cg4(prev + d);
+                n = round_to<A>(n);                      // what later tokens and the prompt kernel see
+                st4(prev + d, n);
+                for (int j = 0; j < n_mu; ++j) {
+                    const float4 m = *reinterpret_cast<const float4*>(p.mu + (size_t)j * D + d);
+                    st4(mixed + (size_t)j * p.n_rows * D + d, make_float4(shifted(n.x, b.x, m.x), shifted(n.y, b.y, m.y),
+                                                                          shifted(n.z, b.z, m.z), shifted(n.w, b.w, m.w)));
+                }
+            }
         } else {
-            h[d] = from_f<A>(u_s[d] * inv * (p.w_offset + p.w[d]));
+            const A n = from_f<A>(u_s[d] * inv * (p.w_offset + p.w[d]));
+            h[d] = n;
+            if (n_mu > 0) {
+                const float b = first ? 0.f : ld_cg(prev + d);
+                prev[d] = n;
+                for (int j = 0; j < n_mu; ++j)
+                    mixed[(size_t)j * p.n_rows * D + d] = from_f<A>(shifted(to_f(n), b, p.mu[(size_t)j * D + d]));
+            }
         }
     }
 }
 
-// in place: the square of relu
-template <typename A>
-__global__ void __launch_bounds__(256) relu2_kernel(A* x, long long n) {
+// Inputs of projections that look one token back, for a prompt portion: mixed[j][row] = h + (h_before - h) * mu_j.
+// h_before of a sequence's first row is what earlier calls left in prev (zeros at position 0); the CTA of that row
+// also renews prev, with the last row's h.
+typedef decoder_shift_args ShiftParams;
+
+template <typename A, int V>
+__global__ void __launch_bounds__(256) token_shift_kernel(const ShiftParams p) {
     griddep_launch_dependents();
     griddep_wait();
-    const long long stride = (long long)gridDim.x * blockDim.x;
-    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n / 4; i += stride) {
-        float4 v = ld_cg4(x + 4 * i);
-        v.x = fmaxf(v.x, 0.f), v.y = fmaxf(v.y, 0.f), v.z = fmaxf(v.z, 0.f), v.w = fmaxf(v.w, 0.f);
-        st4(x + 4 * i, make_float4(v.x * v.x, v.y * v.y, v.z * v.z, v.w * v.w));
-    }
-    if (blockIdx.x == 0 && threadIdx.x < (n & 3)) {
-        const long long i = (n & ~3ll) + threadIdx.x;
-        const float v = fmaxf(ld_cg(x + i), 0.f);
-        x[i] = from_f<A>(v * v);
+    const int row = blockIdx.x, b = row / p.T, t = row - b * p.T, D = p.D;
+    const size_t n = (size_t)p.B * p.T * D;
+    const A* h = reinterpret_cast<const A*>(p.h) + (size_t)row * D;
+    const A* last = reinterpret_cast<const A*>(p.h) + ((size_t)b * p.T + p.T - 1) * D;
+    A* prev = reinterpret_cast<A*>(p.prev) + (size_t)b * D;
+    A* mixed = reinterpret_cast<A*>(p.mixed) + (size_t)row * D;
+    const bool first = t == 0 && p.pos[0] == 0;
+    const A* before = t == 0 ? prev : h - D;
+    for (int d = threadIdx.x * V; d < D; d += blockDim.x * V) {
+        if constexpr (V == 4) {
+            const float4 c = ld_cg4(h + d), o = first ? make_float4(0.f, 0.f, 0.f, 0.f) : ld_cg4(before + d);
+            if (t == 0) st4(prev + d, ld_cg4(last + d));
+            for (int j = 0; j < p.n_mu; ++j) {
+                const float4 m = *reinterpret_cast<const float4*>(p.mu + (size_t)j * D + d);
+                st4(mixed + j * n + d, make_float4(shifted(c.x, o.x, m.x), shifted(c.y, o.y, m.y), shifted(c.z, o.z, m.z),
+                                                   shifted(c.w, o.w, m.w)));
+            }
+        } else {
+            const float c = ld_cg(h + d), o = first ? 0.f : ld_cg(before + d);
+            if (t == 0) prev[d] = from_f<A>(ld_cg(last + d));
+            for (int j = 0; j < p.n_mu; ++j) mixed[j * n + d] = from_f<A>(shifted(c, o, p.mu[(size_t)j * D + d]));
+        }
     }
 }
 

@@ -1,4 +1,4 @@
-// Dense bf16 linear for decode-sized batches (up to 8 rows) on sm_100a: out[m][n] = act(sum_k W[n][k] x[m][k]).
+// Dense bf16 linear for decode-sized batches (up to 8 rows) on sm_100a: out[m][n] = act(sum_k W[n][k] x[m][k] + bias[n]).
 //
 // HBM-bound: W is read exactly once.  A CTA owns 16 rows of W; its eight warps split K, each streaming its
 // slice with one 128-bit load per lane and row (lane (g, q) of the MMA holds rows g and g+8, 8 consecutive k
@@ -6,8 +6,12 @@
 // those registers, as in lm_head.cuh).  The first kRowsPre k-steps of W are requested before the wait for the
 // previous kernel of the stream, so the weights' latency runs underneath its tail.  The rows of x are the
 // MMA's N = 8 and come from L2.  Warp partials meet in shared memory in a fixed order.
+// W may consist of segments of rows with an input each (projections of one token's differently mixed inputs in one
+// launch).  Gated feed-forwards: W holds blocks of 8 gate and 8 up rows, so a CTA makes 8 activations.
 #pragma once
 #include "decoder_common.cuh"
+#include "decoder_ops.h"
+#include "gate.cuh"
 #include "lm_head.cuh"
 
 namespace tsp {
@@ -15,13 +19,7 @@ namespace tsp {
 constexpr int kRowsWarps = 8;
 constexpr int kRowsPre = 6;   // k-steps of 32 whose weights are in flight per warp: what two CTAs per SM have registers for
 
-struct RowsLinearParams {
-    const bf16* x;     // [M][K]
-    const bf16* w;     // [N][K]
-    void* out;         // [M][N] bf16 or fp32
-    int M, N, K;       // M <= 8, K a multiple of 8
-    int act;           // 1: square of relu
-};
+typedef decoder_linear_args RowsLinearParams;
 
 template <typename O>
 __global__ void __launch_bounds__(kRowsWarps * 32, 2) rows_linear_kernel(const RowsLinearParams p) {
@@ -33,9 +31,11 @@ __global__ void __launch_bounds__(kRowsWarps * 32, 2) rows_linear_kernel(const R
     const int n0 = blockIdx.x * 16;
     const int s0 = steps * warp / kRowsWarps, s1 = steps * (warp + 1) / kRowsWarps;
     const bool ok0 = n0 + g < p.N, ok1 = n0 + g + 8 < p.N;
-    const bf16* w0 = p.w + (size_t)(ok0 ? n0 + g : 0) * K + q * 8;
-    const bf16* w1 = p.w + (size_t)(ok1 ? n0 + g + 8 : 0) * K + q * 8;
-    const bf16* x = p.x + (size_t)(g < p.M ? g : 0) * K + q * 8;
+    const bf16* w = reinterpret_cast<const bf16*>(p.w);
+    const bf16* w0 = w + (size_t)(ok0 ? n0 + g : 0) * K + q * 8;
+    const bf16* w1 = w + (size_t)(ok1 ? n0 + g + 8 : 0) * K + q * 8;
+    const int seg = p.seg_rows > 0 ? min(n0 / p.seg_rows, p.n_seg - 1) : 0;
+    const bf16* x = reinterpret_cast<const bf16*>(p.x) + (size_t)seg * p.M * K + (size_t)(g < p.M ? g : 0) * K + q * 8;
     const bool xok = g < p.M;
     const uint4 zero = make_uint4(0, 0, 0, 0);
     uint4 a[kRowsPre], b[kRowsPre];
@@ -65,11 +65,16 @@ __global__ void __launch_bounds__(kRowsWarps * 32, 2) rows_linear_kernel(const R
     __syncthreads();
     if (tid < 128) {
         const int r = tid & 15, t = tid >> 4;
-        if (t < p.M && n0 + r < p.N) {
-            float v = 0.f;
+        float v = 0.f;
 #pragma unroll
-            for (int i = 0; i < kRowsWarps; ++i) v += part[i][r][t];
-            if (p.act == 1) v = fmaxf(v, 0.f), v *= v;
+        for (int i = 0; i < kRowsWarps; ++i) v += part[i][r][t];
+        const bool live = t < p.M && n0 + r < p.N;
+        if (p.bias && n0 + r < p.N) v += p.bias[n0 + r];
+        if (p.gate.kind) {
+            const float up = __shfl_down_sync(0xffffffffu, v, 8);
+            if (live && r < 8) reinterpret_cast<O*>(p.out)[(size_t)t * (p.N / 2) + n0 / 2 + r] = from_f<O>(gated(v, up, p.gate));
+        } else if (live) {
+            if (p.relu2) v = fmaxf(v, 0.f), v *= v;
             reinterpret_cast<O*>(p.out)[(size_t)t * p.N + n0 + r] = from_f<O>(v);
         }
     }

@@ -15,13 +15,11 @@
 // under the other's sigmoids.  Roles: warp 0 TMA, warp 1 MMA issue and tensor memory, warps 2-9 weights (one
 // 32-lane quarter of tensor memory and one half of the keys each) and the gated output.  Every wait is bounded.
 #pragma once
-#include "delta_rule.cuh"
+#include "decoder_status.cuh"
 #include "sigmoid_attn.cuh"
 #include "tcgen05_sm100.cuh"
 
 namespace tsp {
-
-__device__ int g_decoder_status = 0;   // set by a kernel whose bounded wait ran out
 
 struct AttnTcSmem {
     static constexpr int threads = 320;
@@ -31,24 +29,6 @@ struct AttnTcSmem {
     static constexpr int data = 1024;
     static int total(int qk_blocks, int v_blocks) { return 1024 + data + (2 * qk_blocks + v_blocks) * block; }
 };
-
-__device__ __forceinline__ float ex2_approx(float x) {
-    float y;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
-__device__ __forceinline__ float rcp_approx(float x) {
-    float y;
-    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
-__device__ __forceinline__ float2 add2(float2 a, float2 b) {
-    float2 d;
-    asm("add.rn.f32x2 %0, %1, %2;"
-        : "=l"(reinterpret_cast<unsigned long long&>(d))
-        : "l"(reinterpret_cast<const unsigned long long&>(a)), "l"(reinterpret_cast<const unsigned long long&>(b)));
-    return d;
-}
 
 // 1 / (1 + 2^x) of four values with one reciprocal
 __device__ __forceinline__ void sigmoid4(float2 x01, float2 x23, float (&w)[4]) {

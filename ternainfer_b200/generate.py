@@ -57,12 +57,12 @@ class FastGen:
         s = torch.cuda.Stream()
         s.wait_stream(torch.cuda.current_stream())
         with torch.cuda.stream(s):          # warm-up forwards outside capture (one-time library set-up)
-            self.model(self._prefill_tokens, self.cache, self._prefill_pos, greedy_last=True)
+            self.model(self._prefill_tokens, self.cache, self._prefill_pos, greedy_last=True, start=0)
             self.model(self._tokens, self.cache, self._pos, greedy_last=True)
         torch.cuda.current_stream().wait_stream(s)
         self._prefill_graph = torch.cuda.CUDAGraph()
         with torch.cuda.graph(self._prefill_graph):
-            self._prefill_next = self.model(self._prefill_tokens, self.cache, self._prefill_pos, greedy_last=True)
+            self._prefill_next = self.model(self._prefill_tokens, self.cache, self._prefill_pos, greedy_last=True, start=0)
         self._decode_graph = torch.cuda.CUDAGraph()
         with torch.cuda.graph(self._decode_graph):
             self._decode_next = self.model(self._tokens, self.cache, self._pos, greedy_last=True)
@@ -81,7 +81,7 @@ class FastGen:
             self._prefill_graph.replay()
             nxt = self._prefill_next
         else:
-            nxt = self.model(self._prefill_tokens, self.cache, self._prefill_pos, greedy_last=True)
+            nxt = self.model(self._prefill_tokens, self.cache, self._prefill_pos, greedy_last=True, start=0)
         torch.cuda.synchronize()
         t1 = time.perf_counter()
         for i in range(a.gen_length):
@@ -167,7 +167,7 @@ class StepEngine:
             return logits
         logits = self.model(torch.tensor([tokens], device=self.device), r.cache,
                             torch.arange(start, r.length, device=self.device),
-                            want=torch.tensor(want or [len(tokens) - 1], device=self.device))
+                            want=torch.tensor(want or [len(tokens) - 1], device=self.device), start=start)
         if not want:
             return None
         _check_status(self.model)

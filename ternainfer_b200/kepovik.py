@@ -173,10 +173,10 @@ class Kepovik(nn.Module):
         return SequenceCache(layers, torch.zeros(batch, dtype=torch.int64, device=device))
 
     def forward(self, tokens: torch.Tensor, cache: SequenceCache, pos: torch.Tensor, greedy_last: bool = False,
-                want: Optional[torch.Tensor] = None, on_layer=None):
+                want: Optional[torch.Tensor] = None, start: Optional[int] = None, on_layer=None):
         """tokens [B, T]; pos [T] (device int64, consecutive).  fp32 logits [B, T, vocab], or [B, len(want), vocab] at
         the places ``want`` (device int64) among the T, or with ``greedy_last`` the greedy token after every
-        sequence's last position, int64 [B].  ``on_layer(i, x)`` is called with the streams after layer i."""
+        sequence's last position, int64 [B].  ``start``: pos[0] as the host knows it (not needed here).  ``on_layer(i, x)`` is called with the streams after layer i."""
         a = self.args
         B, T = tokens.shape
         step = T == 1

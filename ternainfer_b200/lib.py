@@ -1,13 +1,13 @@
-"""ctypes bindings of ``libternaspmm.so`` and ``libdecoderops.so`` (built in-tree under ``csrc/``).
+"""ctypes bindings of ``libternaspmm.so`` and the dense decoders' libraries (built in-tree under ``csrc/``).
 
 The reference binds its library with ``ctypes.CDLL('./kernels/libternaspmm.so')``
 and passes every pointer as ``c_void_p`` (model.py:21, :76-89 of
 Gu-J/TernaInfer); this module does the same against the B200 library and
 declares argument types so that mistakes fail in Python rather than on the GPU.
 There is no fallback: if the library is missing, loading raises.
-``libdecoderops.so`` (include/decoder_ops.h) holds the kernels of the dense
-decoders; its calls take argument structs and return a status, which
-``check`` turns into an exception.
+The libraries of the dense decoders (include/decoder_ops.h) are loaded one by
+one, at the first call into each; their calls take argument structs and return
+a status, which ``check`` turns into an exception.
 """
 from __future__ import annotations
 
@@ -19,7 +19,6 @@ import subprocess
 _HERE = os.path.dirname(os.path.abspath(__file__))
 _CSRC = os.path.join(_HERE, "csrc")
 _LIB = None
-_DECODER_LIB = None
 
 _P = ctypes.c_void_p
 _I = ctypes.c_int
@@ -33,46 +32,61 @@ class ListItem(ctypes.Structure):
                [(n, _I) for n in ("ws_num", "M", "N", "K", "seg1", "seg2", "seg3", "prefill_form")]
 
 
+class Gate(ctypes.Structure):
+    """``decoder_gate``: activation of a gated feed-forward."""
+    _fields_ = [("kind", _I), ("alpha", ctypes.c_float), ("limit", ctypes.c_float)]
+
+
 def _struct(name, fields):
     """``fields``: 'type: names' lines in the order of the C struct."""
-    kinds = {"p": _P, "i": _I, "l": ctypes.c_longlong, "f": ctypes.c_float}
+    kinds = {"p": _P, "i": _I, "l": ctypes.c_longlong, "f": ctypes.c_float, "g": Gate}
     flat = [(n, kinds[line[0]]) for line in fields for n in line[2:].split()]
     return type(name, (ctypes.Structure,), {"_fields_": flat})
 
 
 # the argument structs of include/decoder_ops.h
 EmbedArgs = _struct("EmbedArgs", ["p tokens pos prev embed bigram x", "l mul_prev mul_cur buckets", "i B T S D V"])
-HyperArgs = _struct("HyperArgs", ["p x y mix out in_ w rows h", "f m w_offset eps", "i D S n_rows"])
+HyperArgs = _struct("HyperArgs", ["p x y mix out in_ w rows h y2 slots slot_w mu prev mixed pos", "f m w_offset eps",
+                                  "i D S n_rows top n_mu"])
+ShiftArgs = _struct("ShiftArgs", ["p h prev mu mixed pos", "i B T D n_mu"])
+LinearArgs = _struct("LinearArgs", ["p x w bias out", "i M N K relu2 seg_rows n_seg", "g gate"])
 DeltaArgs = _struct("DeltaArgs", ["p proj zw w2 w0 a_bias norm pos state o y", "i B T H dk dv rank", "l ld",
                                   "i off_r off_k off_v off_a off_g off_w1", "f eps"])
 AttnArgs = _struct("AttnArgs", ["p proj ck cv q_norm k_norm bias slope pos y", "i B T H G dim vdim", "l ld",
                                 "i off_q off_k off_v off_g", "i chunk slots", "f scale eps"])
+WkvArgs = _struct("WkvArgs", ["p r k v g t1 zw w2 w0 u norm pos state part o y", "i B T H dk dv rank", "l ld ld_t", "i n_seg seg_len", "f eps"])
+LatentPrepArgs = _struct("LatentPrepArgs", ["p z cq cache q_norm kv_norm trig pos", "i B T slots ld r_at R rot dims q_rank", "l ld_z",
+                                            "i off_q off_kv", "f eps"])
+RotateArgs = _struct("RotateArgs", ["p src dst trig pos", "i B T H rot dims", "l ld_src ld_dst", "i head_src head_dst off_src off_dst"])
+AbsorbArgs = _struct("AbsorbArgs", ["p q w_uk qa trig pos", "i B T H dim rot dims R r_at ld"])
+LatentAttnArgs = _struct("LatentAttnArgs", ["p qa cache sink pos out w_uv part ml y", "i B T H R ld vdim slots splits", "f scale"])
+LatentPromptArgs = _struct("LatentPromptArgs", ["p q kv cache sink y", "i B T H dim rot vdim slots ld r_at start off_v", "l ld_kv", "f scale"])
+MoeArgs = _struct("MoeArgs", ["p logits router_bias chosen weight counts rank slots x sorted w_up act w_down w_rest rest bias out",
+                              "i M E top K ff D K_rest", "g gate"])
+GroupGemmArgs = _struct("GroupGemmArgs", ["p a w bias counts out", "i rows groups N K", "g gate"])
 
 
 def library_path() -> str:
     return os.path.join(_CSRC, "libternaspmm.so")
 
 
-def decoder_library_path() -> str:
-    return os.path.join(_CSRC, "libdecoderops.so")
-
-
-def build_library(verbose: bool = False) -> str:
+def build_library(target: str = "all", verbose: bool = False) -> str:
     """Compile the libraries for sm_100a with nvcc (``make -C csrc``)."""
-    subprocess.run(["make", "-C", _CSRC] + (["verbose"] if verbose else []), check=True)
+    subprocess.run(["make", "-C", _CSRC, "verbose" if verbose else target], check=True, stdout=None if verbose else subprocess.DEVNULL)
     return library_path()
 
 
-def build_decoder_library() -> str:
-    """Compile ``libdecoderops.so`` alone, if it is not up to date; safe to call from several processes."""
+def build_decoder_library(*names: str):
+    """Compile the dense decoders' libraries of these names (all without any), as far as they are not up to date; safe to
+    call from several processes."""
+    files = [f"lib{n}.so" for n in names or DECODER_LIBRARIES]
     with open(os.path.join(_CSRC, "Makefile")) as lock:
         fcntl.flock(lock, fcntl.LOCK_EX)
-        subprocess.run(["make", "-C", _CSRC, "libdecoderops.so"], check=True, stdout=subprocess.DEVNULL)
-    return decoder_library_path()
+        subprocess.run(["make", "-j", str(len(files)), "-C", _CSRC] + files, check=True, stdout=subprocess.DEVNULL)
 
 
 class DecoderOpsError(RuntimeError):
-    """A call into ``libdecoderops.so`` was refused; the library has written the reason to stderr."""
+    """A call into a dense decoders' library was refused; the library has written the reason to stderr."""
 
 
 def check(status: int):
@@ -80,38 +94,59 @@ def check(status: int):
         raise DecoderOpsError({1: "shape not supported", 2: "bad pointer", 3: "launch failed", 4: "a wait inside a kernel ran out"}.get(status, str(status)))
 
 
-def load_decoder_library() -> ctypes.CDLL:
-    """Load ``libdecoderops.so``; raises ``OSError`` if it has not been built."""
-    global _DECODER_LIB
-    if _DECODER_LIB is not None:
-        return _DECODER_LIB
-    path = decoder_library_path()
-    if not os.path.exists(path):
-        raise OSError(f"{path} not found: build it with `make -C {_CSRC} libdecoderops.so` (or __graft_entry__.build())")
-    lib = ctypes.CDLL(path)
-    L = ctypes.c_longlong
-    for name, args in (("decoder_embed", [ctypes.POINTER(EmbedArgs), _I, _I, _P]),
-                       ("decoder_hyper", [ctypes.POINTER(HyperArgs), _I, _I, _P]),
-                       ("decoder_rows_linear", [_P, _P, _P, _I, _I, _I, _I, _I, _I, _P]),
-                       ("decoder_head_argmax", [_P, _P, _I, _I, _I, _P, _P, _P, _P]),
-                       ("decoder_relu2", [_P, L, _I, _I, _P]),
-                       ("decoder_delta", [ctypes.POINTER(DeltaArgs), _I, _I, _P]),
-                       ("decoder_tanh_cols", [_P, L, _I, _I, L, _P, _I, _I, _P]),
-                       ("decoder_attn", [ctypes.POINTER(AttnArgs), _I, _I, _I, _P])):
-        fn = getattr(lib, name)
-        fn.argtypes = args
-        fn.restype = _I
-    lib.decoder_head_scratch_bytes.argtypes = []
-    lib.decoder_head_scratch_bytes.restype = L
-    lib.decoder_status.argtypes = []
-    lib.decoder_status.restype = _I
-    _DECODER_LIB = lib
-    return lib
+_L = ctypes.c_longlong
 
 
-DECODER_SYMBOLS = ("decoder_embed", "decoder_hyper", "decoder_rows_linear", "decoder_head_scratch_bytes",
-                   "decoder_head_argmax", "decoder_relu2", "decoder_delta", "decoder_tanh_cols", "decoder_attn",
-                   "decoder_status")
+def _calls(*calls):
+    """name -> argument types: a struct first (by reference), or the list as it is."""
+    return {name: ([ctypes.POINTER(args[0])] + args[1:] if isinstance(args[0], type(ctypes.Structure)) else args) if args else []
+            for name, args in calls}
+
+
+# library -> entry points and their argument types; everything returns int but for the names in _LONG
+DECODER_LIBRARIES = {
+    "decoderops": _calls(("decoder_embed", [EmbedArgs, _I, _I, _P]), ("decoder_hyper", [HyperArgs, _I, _I, _P]),
+                         ("decoder_token_shift", [ShiftArgs, _I, _I, _P]), ("decoder_rows_linear", [LinearArgs, _I, _I, _P]),
+                         ("decoder_gated", [_P, _P, _P, _L, _I, ctypes.POINTER(Gate), _I, _I, _P]),
+                         ("decoder_head_argmax", [_P, _P, _I, _I, _I, _P, _P, _P, _P]), ("decoder_head_scratch_bytes", []),
+                         ("decoder_relu2", [_P, _L, _I, _I, _P]), ("decoder_tanh_cols", [_P, _L, _I, _I, _L, _P, _I, _I, _P])),
+    "deltaops": _calls(("decoder_delta", [DeltaArgs, _I, _I, _P]), ("decoder_attn", [AttnArgs, _I, _I, _I, _P]), ("decoder_status", [])),
+    "latentops": _calls(("decoder_wkv", [WkvArgs, _I, _I, _P]), ("decoder_latent_prep", [LatentPrepArgs, _I, _I, _P]),
+                        ("decoder_rotate", [RotateArgs, _I, _I, _P]), ("decoder_absorb", [AbsorbArgs, _I, _P]),
+                        ("decoder_latent_attn", [LatentAttnArgs, _I, _I, _P]), ("decoder_latent_step", [LatentAttnArgs, _I, _P]),
+                        ("decoder_latent_step_width", []), ("decoder_latent_prompt", [LatentPromptArgs, _P]),
+                        ("decoder_moe_route", [MoeArgs, _I, _P]), ("decoder_moe_plain", [MoeArgs, _I, _I, _P]),
+                        ("decoder_moe_up_step", [MoeArgs, _I, _P]), ("decoder_moe_down_step", [MoeArgs, _I, _P]),
+                        ("decoder_group_gemm", [GroupGemmArgs, _P]), ("decoder_latent_status", [])),
+}
+_LONG = ("decoder_head_scratch_bytes",)
+DECODER_SYMBOLS = tuple(s for calls in DECODER_LIBRARIES.values() for s in calls)
+
+
+class _DecoderLibrary:
+    """The entry points of all dense decoders' libraries; each library is loaded at the first call into it."""
+
+    def __getattr__(self, symbol):
+        for name, calls in DECODER_LIBRARIES.items():
+            if symbol in calls:
+                path = os.path.join(_CSRC, f"lib{name}.so")
+                if not os.path.exists(path):
+                    raise OSError(f"{path} not found: build it with `make -C {_CSRC} lib{name}.so` (or __graft_entry__.build())")
+                lib = ctypes.CDLL(path)
+                for s, args in calls.items():
+                    fn = getattr(lib, s)
+                    fn.argtypes, fn.restype = args, _L if s in _LONG else _I
+                    setattr(self, s, fn)
+                return getattr(self, symbol)
+        raise AttributeError(symbol)
+
+
+_DECODER_LIB = _DecoderLibrary()
+
+
+def load_decoder_library() -> _DecoderLibrary:
+    """The dense decoders' entry points; calling one raises ``OSError`` if its library has not been built."""
+    return _DECODER_LIB
 
 
 def load_library() -> ctypes.CDLL:

@@ -264,10 +264,10 @@ class Transformer(nn.Module):
         return (None, logits.argmax(-1)) if greedy else logits
 
     def forward(self, tokens: torch.Tensor, cache: List[LayerCache], pos: torch.Tensor, greedy_last: bool = False,
-                want: Optional[torch.Tensor] = None):
+                want: Optional[torch.Tensor] = None, start: Optional[int] = None):
         """tokens [B, T]; pos [T] (device int64) = positions written in the cache.
         Returns fp32 logits [B, T, vocab] (model.py:380-386 of the reference), or [B, len(want), vocab]
-        at the places ``want`` (device int64) among the T; with ``greedy_last`` only the greedy token of every sequence's last position, int64 [B] (what the generation
+        at the places ``want`` (device int64) among the T (``start``, the host's copy of pos[0], is not needed here); with ``greedy_last`` only the greedy token of every sequence's last position, int64 [B] (what the generation
         loop needs: generate.py:274, :283, :305 of the reference)."""
         if self._rope is None or self._rope[0].device != tokens.device:
             self._rope = rope_tables(self.args.head_dim, self.max_seq_len, self.args.rope_theta, tokens.device)

@@ -46,12 +46,8 @@ def main() -> int:
     ap.add_argument("--max-tokens", type=int, required=True, help="most tokens that live requests hold at any time")
     a = ap.parse_args()
     import torch
-    from .lib import build_decoder_library, build_library
-    from .registry import UnsupportedDtype, load_model, read_config
-    if read_config(a.model).get("architecture") == "TernaInfer":
-        build_library()
-    else:
-        build_decoder_library()
+    from .registry import UnsupportedDtype, build_libraries, load_model
+    build_libraries(a.model)
     from .generate import StepEngine
     try:
         model = load_model(a.model, getattr(torch, a.dtype), max(1, a.max_tokens))

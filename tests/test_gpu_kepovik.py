@@ -3,6 +3,7 @@
 Random weights hide a wrong key among hundreds, so the attention tests give chosen keys and queries one large
 common component: the chosen key's weight is then near one and its value dominates the output, and a key that
 must not be seen would dominate it just as visibly."""
+import ctypes
 import json
 import os
 import subprocess
@@ -351,14 +352,14 @@ def test_linear_with_and_without_squared_relu(dec, M, N, K):
 
 def test_bad_calls_are_refused_on_the_host(dec):
     from ternainfer_b200 import decoder_ops as ops
-    from ternainfer_b200.lib import DecoderOpsError
+    from ternainfer_b200.lib import DecoderOpsError, LinearArgs
     with pytest.raises(RuntimeError):
         ops.linear(torch.zeros((1, 8)), torch.zeros((1, 8)))
     with pytest.raises(DecoderOpsError):
         x = torch.zeros((1, 9, 16), device="cuda")          # nine streams
         ops.hyper_norm(x, torch.zeros(16, device="cuda"), 1e-5, torch.float32)
-    assert dec.decoder_rows_linear(None, None, None, 1, 1, 8, 0, 0, 0, None) == 2
-    assert dec.decoder_rows_linear(None, None, None, 9, 1, 8, 0, 0, 0, None) == 1
+    assert dec.decoder_rows_linear(ctypes.byref(LinearArgs(M=1, N=1, K=8)), 0, 0, None) == 2
+    assert dec.decoder_rows_linear(ctypes.byref(LinearArgs(M=9, N=1, K=8)), 0, 0, None) == 1
 
 
 # ------------------------------------------------------------------------------- the model

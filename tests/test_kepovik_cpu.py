@@ -98,7 +98,7 @@ class Echo:
     def make_cache(self, batch, device):
         return [torch.zeros(self.max_seq_len, dtype=torch.long)]
 
-    def __call__(self, toks, cache, pos, greedy_last=False, want=None):
+    def __call__(self, toks, cache, pos, greedy_last=False, want=None, start=None):
         cache[0][pos] = toks[0]
         out = torch.stack([torch.stack([cache[0][:p + 1].sum(), p]) for p in pos]).float()[None]
         return out if want is None else out[:, want]
@@ -165,16 +165,15 @@ def test_decoder_library_exports_what_its_header_declares():
 def test_argument_structs_match_the_header():
     from ternainfer_b200 import lib as L
     text = re.sub(r"/\*.*?\*/", "", open(os.path.join(ROOT, "include", "decoder_ops.h")).read(), flags=re.S)
-    size = {"int": 4, "float": 4, "long long": 8}
+    size = {"int": 4, "float": 4, "long long": 8, "decoder_gate": 12}
     for body, name in re.findall(r"typedef struct \{(.*?)\} (decoder_\w+);", text, flags=re.S):
-        cls = {"decoder_embed_args": L.EmbedArgs, "decoder_hyper_args": L.HyperArgs, "decoder_delta_args": L.DeltaArgs,
-               "decoder_attn_args": L.AttnArgs}[name]
+        cls = getattr(L, "".join(w.capitalize() for w in name.split("_")[1:]))
         fields = []
         for line in body.split(";"):
             line = line.strip()
             if not line:
                 continue
-            m = re.match(r"(?:const )?(void|float|int|long long)\s*(\*?)\s*(.*)", line)
+            m = re.match(r"(?:const )?(void|float|int|long long|decoder_gate)\s*(\*?)\s*(.*)", line)
             for f in m.group(3).split(","):
                 fields.append((f.strip(), 8 if m.group(2) else size[m.group(1)]))
         got = [(n.rstrip("_"), ctypes.sizeof(t)) for n, t in cls._fields_]
