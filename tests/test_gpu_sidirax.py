@@ -1,0 +1,758 @@
+"""GPU: the kernels of the Sidirax decoder and the model on them against the plain CPU restatement.
+
+Random weights hide a wrong key among hundreds, so the attention tests give chosen queries a large component along
+chosen keys: the chosen key's weight is then near one and its value dominates the output, and a key that must not be
+seen would dominate it just as visibly."""
+import ctypes
+import json
+import os
+import subprocess
+import sys
+
+import numpy as np
+import pytest
+import torch
+
+import sidirax_oracle as o
+from kepovik_util import rel_rms, save_model
+from sidirax_util import CONFIGS, YARN, config, dense, latent, moe, row_errors, tokens, weights, wkv
+
+pytestmark = pytest.mark.gpu
+ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+TOL = {torch.float32: 2e-5, torch.bfloat16: 1.5e-2}
+DTYPES = [torch.float32, torch.bfloat16]
+
+
+@pytest.fixture(scope="module")
+def dec():
+    from ternainfer_b200.lib import build_decoder_library, load_decoder_library
+    build_decoder_library("decoderops", "latentops")
+    torch.backends.cuda.matmul.allow_bf16_reduced_precision_reduction = False
+    lib = load_decoder_library()
+    lib.decoder_latent_status()
+    yield lib
+    assert lib.decoder_latent_status() == 0
+
+
+def cuts(T, sizes):
+    """Portions of the given sizes, over and over, until T tokens are covered."""
+    out, at, i = [], 0, 0
+    while at < T:
+        n = min(sizes[i % len(sizes)], T - at)
+        out.append((at, at + n))
+        at, i = at + n, i + 1
+    return out
+
+
+def singles(a, b):
+    return [(i, i + 1) for i in range(a, b)]
+
+
+def pos(a, b):
+    return torch.arange(a, b, device="cuda")
+
+
+# ------------------------------------------------------------------------------- attention over a latent
+
+def attn_case(H, dim, rot, vdim, R, T, dtype, B=1, seed=0, stand_out=(), scale=None, sink=None):
+    """Queries, latents and shared key parts.  stand_out: (query, key) places; the query gets a large component along
+    that key, in every head of sequence 0, and the key's latent a large one that shows in its value."""
+    g = torch.Generator().manual_seed(seed)
+    n = lambda *s: torch.randn(s, generator=g)
+    q, c, kr = n(B, T, H, dim + rot), n(B, T, R), n(B, T, rot)
+    uk, uv = n(H * dim, R) / R ** 0.5, n(H * vdim, R) / R ** 0.5
+    for i, j in stand_out:
+        c[0, j] *= 2
+    uk, c, kr = uk.to(dtype), c.to(dtype), kr.to(dtype)
+    for i, j in stand_out:
+        k = torch.cat([(uk.float() @ c[0, j].float()).view(H, dim), kr[0, j].float().expand(H, rot)], -1)
+        q[0, i] = 0.3 * q[0, i] + 40 * k / (k * k).sum(-1, keepdim=True) / (scale or (dim + rot) ** -0.5)
+    return dict(q=q.to(dtype), c=c, kr=kr, uk=uk, uv=uv.to(dtype), sink=n(H) if sink is None else torch.full((H,), float(sink)),
+                scale=(dim + rot) ** -0.5 if scale is None else scale, dims=(H, dim, rot, vdim, R))
+
+
+def attn_want(case, causal=None):
+    H, dim, rot, vdim, R = case["dims"]
+    B, T = case["q"].shape[:2]
+    out = []
+    for b in range(B):
+        c = case["c"][b].double()
+        k = torch.cat([(c @ case["uk"].double().T).view(T, H, dim), case["kr"][b].double()[:, None].expand(T, H, rot)], -1)
+        v = (c @ case["uv"].double().T).view(T, H, vdim)
+        s = torch.einsum("ihd,jhd->hij", case["q"][b].double(), k) * case["scale"]
+        s = s.masked_fill(~(torch.ones(T, T).tril().bool() if causal is None else causal), -torch.inf)
+        p = torch.softmax(torch.cat([s, case["sink"].double()[:, None, None].expand(H, T, 1)], -1), -1)[..., :T]
+        out.append(torch.einsum("hij,jhd->ihd", p, v).flatten(1))
+    return torch.stack(out)
+
+
+def attn_got(case, parts, slots=None, path=None, stale=3.0, splits=None):
+    """The portions one after the other, every one with its keys appended first; later slots hold stale data."""
+    from ternainfer_b200 import decoder_ops as ops
+    H, dim, rot, vdim, R = case["dims"]
+    B, T = case["q"].shape[:2]
+    dtype = case["q"].dtype
+    r_at = -(-R // 8) * 8
+    ld = -(-(r_at + rot) // 8) * 8
+    cache = torch.full((B, slots or T, ld), stale, dtype=dtype, device="cuda")
+    cache[:, :, R:r_at] = 0
+    cache[:, :, r_at + rot:] = 0
+    uk, uv, sink = case["uk"].cuda(), case["uv"].cuda(), case["sink"].cuda()
+    ys = []
+    for a, b in parts:
+        n = b - a
+        cache[:, a:b, :R], cache[:, a:b, r_at:r_at + rot] = case["c"][:, a:b].cuda(), case["kr"][:, a:b].cuda()
+        q = case["q"][:, a:b].reshape(B * n, -1).contiguous().cuda()
+        kind = path or ("plain" if dtype == torch.float32 else "step" if n <= 8 else "prompt")
+        if kind == "prompt":
+            y = ops.latent_attention_prompt(q, torch.cat([uk, uv]), cache, sink, a, n, H, dim, rot, vdim, r_at, case["scale"])
+        else:
+            qa = ops.absorb(q, uk, H, dim, rot, r_at, ld, None, pos(a, b), n)
+            if kind == "step":
+                y = ops.latent_attention_step(qa, cache, uv, sink, pos(a, b), n, vdim, case["scale"], splits=splits)
+            else:
+                y = ops.latent_attention_plain(qa, cache, uv, sink, pos(a, b), n, vdim, case["scale"])
+        ys.append(y.view(B, n, -1))
+    return torch.cat(ys, 1)
+
+
+SHAPES = [  # H, dim, rot, vdim, R, T
+    (4, 64, 32, 48, 96, 150), (20, 16, 16, 32, 40, 90), (3, 128, 64, 128, 512, 200), (2, 32, 16, 16, 264, 300), (33, 16, 48, 16, 24, 70),
+    (1, 112, 32, 96, 128, 260), (5, 48, 64, 80, 600, 80)]
+ODD = [(3, 12, 6, 9, 21, 70), (2, 7, 5, 11, 33, 40), (1, 200, 24, 130, 16, 150), (2, 16, 16, 16, 1100, 20)]
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("H,dim,rot,vdim,R,T", SHAPES)
+def test_latent_attention_whole_portions_and_single_tokens(dec, H, dim, rot, vdim, R, T, dtype):
+    case = attn_case(H, dim, rot, vdim, R, T, dtype)
+    want = attn_want(case)[0]
+    first = None
+    for parts in ([(0, T)], cuts(T, [37, 2, 5, 64, 3]), cuts(T, [8]), [(0, T // 2)] + singles(T // 2, T)):
+        got = attn_got(case, parts)[0]
+        assert rel_rms(got, want) < TOL[dtype], parts[:4]
+        first = got if first is None else first
+        assert rel_rms(got, first) < TOL[dtype]
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("H,dim,rot,vdim,R,T", ODD)
+def test_latent_attention_of_any_size(dec, H, dim, rot, vdim, R, T, dtype):
+    case = attn_case(H, dim, rot, vdim, R, T, dtype)
+    for parts in ([(0, T)], cuts(T, [9, 2]), singles(0, T)):
+        assert rel_rms(attn_got(case, parts, path="plain")[0], attn_want(case)[0]) < TOL[dtype], parts[:4]
+
+
+def test_latent_attention_far_keys_and_tile_borders(dec):
+    """One key among 700, far away, at tile borders of the kernels (64 keys, 128 queries) and the token itself."""
+    T = 720
+    places = [(700, 0), (701, 63), (702, 64), (703, 127), (704, 128), (639, 511), (640, 512), (719, 1), (127, 0), (128, 64), (511, 511), (705, 705)]
+    rows = [i for i, _ in places]
+    for dtype in DTYPES:
+        case = attn_case(2, 64, 32, 64, 64, T, dtype, stand_out=places)
+        want = attn_want(case)[0]
+        blind = torch.ones(T, T).tril().bool()
+        for i, j in places:
+            blind[i, j] = False
+        assert (row_errors(attn_want(case, blind)[0][rows], want[rows]) > 0.3).all()     # the planted keys decide
+        for parts in ([(0, T)], [(0, 600), (600, 720)], cuts(699, [130]) + singles(699, T), cuts(T, [8]), [(0, 703), (703, 705), (705, T)]):
+            got = attn_got(case, parts, slots=T + 40)[0]
+            assert rel_rms(got[rows], want[rows]) < 2 * TOL[dtype], parts[:3]
+    for splits in (1, 2, 7, 30, 200):                      # more ranges than keys too
+        got = attn_got(case, cuts(T, [8]), splits=splits)[0]
+        assert rel_rms(got[rows], want[rows]) < 2 * TOL[dtype]
+
+
+def test_latent_attention_does_not_see_the_next_token(dec):
+    """Every query would choose the token after it, by far, if it saw it."""
+    T = 200
+    for dtype in DTYPES:
+        case = attn_case(2, 32, 16, 32, 48, T, dtype, stand_out=[(i, i + 1) for i in range(T - 1)])
+        want = attn_want(case)[0]
+        ahead = torch.ones(T, T).tril(1).bool()
+        assert row_errors(attn_want(case, ahead)[0][:-1], want[:-1]).median() > 0.5
+        for parts in ([(0, T)], cuts(T, [33]), cuts(T, [7]), singles(0, T)):
+            assert rel_rms(attn_got(case, parts)[0], want) < 2 * TOL[dtype]
+
+
+@pytest.mark.parametrize("sink", [-40.0, 0.0, 4.0, 30.0])
+def test_the_sink_counts_once_and_is_not_scaled(dec, sink):
+    for dtype in DTYPES:
+        for scale in (0.02, 0.3, -0.2):
+            case = attn_case(3, 32, 16, 16, 40, 150, dtype, sink=sink, scale=scale)
+            want = attn_want(case)[0]
+            for parts in ([(0, 150)], cuts(150, [8]), [(0, 100)] + singles(100, 150)):
+                got = attn_got(case, parts)[0]
+                assert rel_rms(got, want) < 2 * TOL[dtype], (scale, parts[:2])
+
+
+def test_large_scores_move_the_reference_point(dec):
+    """Scores that grow along the sequence by hundreds: the running maximum moves in almost every tile."""
+    T = 400
+    for dtype in DTYPES:
+        case = attn_case(2, 32, 16, 32, 32, T, dtype, scale=1.0, sink=-5.0)
+        case["kr"] = (case["kr"].float() * 0.1 + torch.linspace(0, 4, T)[None, :, None]).to(dtype)
+        case["q"][..., 32:] = case["q"][..., 32:].abs() + 3
+        want = attn_want(case)[0]
+        for parts in ([(0, T)], cuts(T, [100]), cuts(T, [8])):
+            assert rel_rms(attn_got(case, parts)[0], want) < 3 * TOL[dtype]
+
+
+def test_latent_attention_batch_equals_single_sequences(dec):
+    for dtype in DTYPES:
+        case = attn_case(4, 32, 16, 48, 72, 83, dtype, B=3)
+        parts = [(0, 40), (40, 82), (82, 83)]
+        whole = attn_got(case, parts, slots=90)
+        assert rel_rms(whole.flatten(0, 1), attn_want(case).flatten(0, 1)) < TOL[dtype]
+        for b in range(3):
+            one = {k: (v[b:b + 1] if k in ("q", "c", "kr") else v) for k, v in case.items()}
+            assert rel_rms(attn_got(one, parts, slots=90)[0], whole[b]) < TOL[dtype]
+
+
+@pytest.mark.parametrize("rot", [{"dims": 16, "base": 300.0, "scaling": YARN}, {"dims": 16, "base": 500.0}, {"dims": 6, "base": 20.0}])
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_norms_rotation_and_append(dec, rot, dtype):
+    """Far positions too; a layer that shares a latent leaves the cache alone."""
+    from ternainfer_b200 import decoder_ops as ops
+    from ternainfer_b200.sidirax import _parse_rotation
+    R, rd, qr, T, B, H, dim = 20, 16, 12, 9, 2, 3, 5
+    table = _parse_rotation(rot, "test").table(3000).cuda()
+    g = torch.Generator().manual_seed(0)
+    z = torch.randn((B * T, qr + R + rd + 4), generator=g).to(dtype)
+    qn, kn = 1 + torch.randn(qr, generator=g), 1 + torch.randn(R, generator=g)
+    for start in (0, 700, 2991):
+        cache = torch.full((B, 3000, 40), 5.0, dtype=dtype, device="cuda")
+        at = range(start, start + T)
+        cq = ops.latent_prep(z.cuda(), 2, qn.cuda(), pos(start, start + T), T, 1e-3, cache, 2 + qr, kn.cuda(), 24, rd, table)
+        zd = z.double()
+        assert rel_rms(cq, o.rms(zd[:, 2:2 + qr], 1e-3) * qn.double()) < TOL[dtype]
+        for b in range(B):
+            mine = zd[b * T:(b + 1) * T]
+            got = cache[b, start:start + T]
+            assert rel_rms(got[:, :R], o.rms(mine[:, 2 + qr:2 + qr + R], 1e-3) * kn.double()) < TOL[dtype]
+            assert rel_rms(got[:, 24:], o.rotate(mine[:, 2 + qr + R:2 + qr + R + rd], at, rot)) < TOL[dtype]
+            assert (got[:, R:24] == 5).all() and (cache[b, :start] == 5).all() and (cache[b, start + T:] == 5).all()
+        before = cache.clone()
+        again = ops.latent_prep(z.cuda(), 2, qn.cuda(), pos(start, start + T), T, 1e-3)
+        assert torch.equal(again, cq) and torch.equal(before, cache)
+        q = torch.randn((B * T, H * (dim + rd)), generator=g).to(dtype)
+        turned = q.cuda()
+        ops.rotate(turned, turned, H, dim, dim, rd, table, pos(start, start + T), T)
+        qh = q.view(B, T, H, dim + rd).double()
+        want = torch.cat([qh[..., :dim], torch.stack([o.rotate(qh[b, ..., dim:], at, rot) for b in range(B)])], -1)
+        assert rel_rms(turned, want.reshape(B * T, -1)) < TOL[dtype]
+
+
+@pytest.mark.parametrize("M,T", [(1, 1), (8, 1), (6, 3), (8, 8)])
+@pytest.mark.parametrize("dim,R", [(128, 512), (48, 136), (7, 8), (130, 40)])
+def test_absorbed_queries(dec, M, T, dim, R):
+    from ternainfer_b200 import decoder_ops as ops
+    from ternainfer_b200.sidirax import _parse_rotation
+    rot = {"dims": 8, "base": 300.0}
+    g = torch.Generator().manual_seed(0)
+    H, rd, B = 3, 10, M // T
+    q, uk = torch.randn((M, H * (dim + rd)), generator=g).bfloat16(), (torch.randn((H * dim, R), generator=g) / dim ** 0.5).bfloat16()
+    ld = R + 16
+    qa = ops.absorb(q.cuda(), uk.cuda(), H, dim, rd, R, ld, _parse_rotation(rot, "t").table(60).cuda(), pos(31, 31 + T), T).double().cpu()
+    qh = q.view(B, T, H, dim + rd).double()
+    want = torch.einsum("bthd,hdr->bthr", qh[..., :dim], uk.view(H, dim, R).double())
+    assert rel_rms(qa[:, :, :R].reshape(M, -1), want.reshape(M, -1)) < 4e-3
+    turned = torch.stack([o.rotate(qh[b, ..., dim:], range(31, 31 + T), rot) for b in range(B)])
+    assert rel_rms(qa[:, :, R:R + rd].reshape(M, -1), turned.reshape(M, -1)) < 4e-3 and (qa[:, :, R + rd:] == 0).all()
+
+
+# ------------------------------------------------------------------------------- wkv recurrence
+
+def wkv_case(H, d, rank, T, dtype, B=1, seed=0, w0=None):
+    g = torch.Generator().manual_seed(seed)
+    n = H * d
+    z = {k: torch.randn((B, T, n), generator=g).to(dtype) for k in "rkvg"}
+    z["t1"] = torch.randn((B, T, rank), generator=g).to(dtype)
+    return dict(z=z, w2=(torch.randn((n, rank), generator=g) / rank ** 0.5).to(dtype), u=torch.randn((H, d), generator=g),
+                w0=-2 + 2 * torch.randn(n, generator=g) if w0 is None else torch.full((n,), float(w0)), norm=1 + 0.3 * torch.randn(n, generator=g),
+                H=H, d=d, eps=1e-5)
+
+
+def wkv_want(c):
+    H, d = c["H"], c["d"]
+    ys, states = [], []
+    for b in range(c["z"]["k"].shape[0]):
+        f = lambda n: c["z"][n][b].double()
+        head = lambda t: t.view(t.shape[0], H, d)
+        w = head(torch.exp(-torch.exp(torch.tanh(f("t1")) @ c["w2"].double().T + c["w0"].double())))
+        res = [o.wkv(head(f("r"))[:, h], head(f("k"))[:, h], head(f("v"))[:, h], w[:, h], c["u"][h].double()) for h in range(H)]
+        ys.append(o.rms(torch.stack([r[0] for r in res], 1), c["eps"]).flatten(1) * c["norm"].double() * o.silu(f("g")))
+        states.append(torch.stack([r[1] for r in res]))
+    return torch.stack(ys), torch.stack(states)
+
+
+def wkv_got(c, parts, state=None, segments=None):
+    from ternainfer_b200 import decoder_ops as ops
+    B, T, n = c["z"]["k"].shape
+    if state is None:
+        state = torch.full((B, c["H"], c["d"], c["d"]), 3.0, device="cuda")     # what an earlier sequence left
+    full = torch.cat([c["z"][k] for k in ("r", "k", "v", "g", "t1")], -1)
+    full = torch.nn.functional.pad(full, (0, -full.shape[-1] % 8))
+    ys = []
+    for a, b in parts:
+        z = full[:, a:b].reshape(B * (b - a), -1).contiguous().cuda()
+        r, k, v, g, t1 = (z[:, i * n:] for i in range(5))
+        seg = segments(b - a) if segments and b - a > 1 else None
+        y = ops.wkv(r, k, v, g, t1, c["w2"].cuda(), c["w0"].cuda(), c["u"].cuda(), c["norm"].cuda(), state, pos(a, b), b - a, c["eps"],
+                    step=b - a == 1, segments=seg)
+        ys.append(y.view(B, b - a, n))
+    return torch.cat(ys, 1), state
+
+
+def cut16(n, most=100):
+    """Segments of 16 tokens (or more, so that there are at most ``most``)."""
+    length = -(-(-(-n // most)) // 16) * 16
+    return -(-n // length), length
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("H,d,rank,T", [(3, 16, 4, 70), (2, 64, 16, 131), (1, 128, 40, 66), (2, 24, 7, 50), (1, 256, 33, 40), (5, 10, 1, 45),
+                                        (2, 96, 64, 49), (1, 1, 3, 20), (2, 200, 8, 35)])
+def test_wkv_whole_portions_segments_and_single_tokens(dec, H, d, rank, T, dtype):
+    c = wkv_case(H, d, rank, T, dtype)
+    want, S = wkv_want(c)
+    tol = 3e-5 if dtype == torch.float32 else 8e-3
+    for parts, seg in (([(0, T)], None), ([(0, T)], cut16), (cuts(T, [16, 2, 17, 5]), None), (cuts(T, [2]), None), (cuts(T, [33, 3]), cut16),
+                       (singles(0, T), None), ([(0, T - 9)] + singles(T - 9, T), lambda n: cut16(n, 2))):
+        got, state = wkv_got(c, parts, segments=seg)
+        assert rel_rms(got[0].view(T * H, d), want[0].reshape(T * H, d)) < (tol if d > 1 else 10 * tol), parts[:3]
+        assert (state.double().cpu() - S).abs().max() < tol * S.abs().max()
+
+
+@pytest.mark.parametrize("w0", [-30.0, -8.0, 1.5, 6.0])
+def test_wkv_with_extreme_decays(dec, w0):
+    """From a state that forgets nothing to one that forgets everything; no step divides by a decay."""
+    for dtype in DTYPES:
+        c = wkv_case(2, 32, 8, 200, dtype, w0=w0)
+        want, S = wkv_want(c)
+        tol = 1e-4 if dtype == torch.float32 else 1.2e-2
+        for parts, seg in (([(0, 200)], None), ([(0, 200)], cut16), ([(0, 90)] + singles(90, 200), None)):
+            got, state = wkv_got(c, parts, segments=seg)
+            assert torch.isfinite(got).all() and row_errors(got[0], want[0]).max() < tol
+            assert (state.double().cpu() - S).abs().max() < tol * S.abs().max().clamp_min(1e-3)
+
+
+def test_wkv_batch_and_restart(dec):
+    """Three sequences at once equal each alone, and a state that another sequence has filled does not matter."""
+    for dtype in DTYPES:
+        c = wkv_case(2, 32, 8, 85, dtype, B=3)
+        parts = [(0, 70), (70, 84), (84, 85)]
+        for seg in (None, cut16):
+            whole, state = wkv_got(c, parts, segments=seg)
+            again, _ = wkv_got(c, parts, state, segments=seg)
+            assert torch.equal(whole, again)
+            for b in range(3):
+                one = dict(c, z={k: v[b:b + 1] for k, v in c["z"].items()})
+                # (the decay's matrix product may sum in another order for another row count)
+                assert rel_rms(wkv_got(one, parts, segments=seg)[0][0], whole[b]) < (1e-5 if dtype == torch.float32 else 4e-3)
+
+
+def test_wkv_remembers_and_the_bonus_is_the_current_token_alone(dec):
+    """A pair written once and read 200 tokens later with decays near one; its own token sees it through the bonus."""
+    d, T = 32, 220
+    for dtype in DTYPES:
+        c = wkv_case(1, d, 2, T, dtype, w0=-12.0)
+        z = c["z"]
+        g = torch.Generator().manual_seed(5)
+        basis = torch.linalg.qr(torch.randn((d, d), generator=g))[0]
+        key = basis[0]
+        z["k"][0] = (torch.randn((T, d - 1), generator=g) @ basis[1:]).to(dtype)      # all other keys orthogonal to it
+        z["k"][0, 3] = (2 * key).to(dtype)
+        z["r"][0, [3, 4, 50, T - 1]] = (5 * key).to(dtype)
+        z["v"][0, 3] *= 4
+        c["u"][:] = -3.0
+        want, _ = wkv_want(c)
+        gate = lambda t: o.silu(z["g"][0, t].double()) * c["norm"].double()
+        cos = lambda x, y: torch.nn.functional.cosine_similarity(x, y, dim=0).item()
+        for parts, seg in (([(0, T)], None), ([(0, T)], cut16), (cuts(T, [30, 2]), None), ([(0, 3)] + singles(3, T), None)):
+            got = wkv_got(c, parts, segments=seg)[0][0].double().cpu()
+            assert row_errors(got, want[0]).max() < (1e-4 if dtype == torch.float32 else 2e-2)
+            v = z["v"][0, 3].double()
+            assert cos(got[T - 1], v * gate(T - 1)) > 0.9 and cos(got[4], v * gate(4)) > 0.9 and cos(got[3], v * gate(3)) < -0.9
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("D", [64, 42])
+def test_token_shift_in_prompts_and_with_the_norm(dec, dtype, D):
+    """The input before the first token counts as zeros; the last input is kept from call to call and sequence by sequence."""
+    from ternainfer_b200 import decoder_ops as ops
+    g = torch.Generator().manual_seed(0)
+    B, T, n = 3, 11, 5
+    x, w, mu = torch.randn((B, T, D), generator=g), 1 + torch.randn(D, generator=g), torch.rand((n, D), generator=g)
+    h = (o.rms(x.double(), 1e-4) * w.double()).to(dtype).double()
+    want = torch.stack([torch.stack([o.token_shift(h[b], m.double()) for b in range(B)]) for m in mu])
+    for parts in ([(0, T)], cuts(T, [1]), cuts(T, [4, 1, 2])):
+        prev = torch.full((B, D), 7.0, dtype=dtype, device="cuda")
+        got = []
+        for a, b in parts:
+            rows = x[:, a:b].reshape(-1, 1, D).contiguous().cuda()
+            if b - a == 1:
+                out = ops.hyper_norm(rows, w.cuda(), 1e-4, dtype, shift=(mu.cuda(), prev, pos(a, b)), step=True)
+                assert rel_rms(out[n], h[:, a]) < TOL[dtype] / 2
+                got.append(out[:n].view(n, B, 1, D))
+            else:
+                hn = ops.hyper_norm(rows, w.cuda(), 1e-4, dtype)
+                got.append(ops.token_shift(hn, mu.cuda(), prev, pos(a, b), b - a).view(n, B, b - a, D))
+        assert rel_rms(torch.cat(got, 2).flatten(0, 2), want.flatten(0, 2)) < TOL[dtype]
+        assert rel_rms(prev, h[:, -1]) < TOL[dtype] / 2
+
+
+# ------------------------------------------------------------------------------- residual, feed-forwards, experts
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("D", [48, 30])
+def test_residual_takes_two_outputs_and_gathered_rows(dec, dtype, D):
+    from ternainfer_b200 import decoder_ops as ops
+    g = torch.Generator().manual_seed(0)
+    M, top = 6, 3
+    x, w = torch.randn((M, 1, D), generator=g), torch.randn(D, generator=g)
+    y, y2, ye = (torch.randn((r, D), generator=g).to(dtype) for r in (M, M, M * top))
+    slots = torch.randperm(M * top, generator=g).view(M, top).int()
+    sw = torch.rand((M, top), generator=g)
+    for kw, add in (({"y2": y2.cuda()}, y2.double()), ({}, 0),
+                    ({"y2": ye.cuda(), "slots": slots.cuda(), "slot_w": sw.cuda()}, (ye.double()[slots.long()] * sw.double()[..., None]).sum(1))):
+        xd = x.clone().cuda()
+        new = x[:, 0].double() + y.double() + add
+        pick = torch.tensor([4, 1], device="cuda")
+        some = ops.hyper_norm(xd, w.cuda(), 1e-5, dtype, y=y.cuda(), rows=pick, **kw)
+        assert torch.equal(xd.cpu(), x) and rel_rms(some, (o.rms(new, 1e-5) * w.double())[[4, 1]]) < TOL[dtype]
+        h = ops.hyper_norm(xd, w.cuda(), 1e-5, dtype, y=y.cuda(), **kw)
+        assert rel_rms(xd[:, 0], new) < 1e-6 and rel_rms(h, o.rms(new, 1e-5) * w.double()) < TOL[dtype]
+
+
+def ff_weights(cfg, D, dtype, seed=0, spread=1.0):
+    g = torch.Generator().manual_seed(seed)
+    n = lambda *s: torch.randn(s, generator=g)
+    ff = cfg["ff"] if cfg["kind"] == "dense" else cfg["expert"]["ff"]
+    if cfg["kind"] == "dense":
+        w = {"gate": n(ff, D) / D ** 0.5, "up": n(ff, D) / D ** 0.5, "down": n(D, ff) / ff ** 0.5, "gate.b": n(ff), "up.b": n(ff), "down.b": n(D)}
+    else:
+        E = cfg["router"]["experts"]
+        w = {"router": spread * n(E, D) / D ** 0.5, "router.b": spread * n(E)}
+        for e in range(E):
+            w.update({f"e{e}.gate": n(ff, D) / D ** 0.5, f"e{e}.up": n(ff, D) / D ** 0.5, f"e{e}.down": n(D, ff) / ff ** 0.5})
+    return {k: v.to(dtype) for k, v in w.items()}
+
+
+def ff_module(cfg, w, dtype):
+    from ternainfer_b200 import decoder_ops as ops
+    from ternainfer_b200.mixers import ExpertFeedForward, GatedFeedForward
+    if cfg["kind"] == "dense":
+        return GatedFeedForward(ops.clamped_gate(1.702, cfg["limit"]), w, dtype).cuda()
+    return ExpertFeedForward(cfg["router"]["experts"], cfg["router"]["top"], ops.silu_gate(), w, dtype).cuda()
+
+
+def ff_total(out):
+    """What the residual would receive."""
+    y = out["y"].double()
+    if "slots" in out:
+        return y + (out["y2"].double()[out["slots"].long()] * out["slot_w"].double()[..., None]).sum(1)
+    return y + out["y2"].double() if "y2" in out else y
+
+
+FFS = [dense(56, 0.8), dense(30, 3.0), dense(264, 1.5), moe(5, 2, 24), moe(4, 4, 40), moe(7, 1, 13), moe(40, 6, 16), moe(3, 2, 300), moe(300, 32, 8)]
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("cfg", FFS, ids=lambda c: "-".join(str(x) for v in c.values() for x in (v.values() if isinstance(v, dict) else [v])))
+def test_feed_forwards(dec, cfg, dtype):
+    """Few rows and many, with another product in the same residual update and without, widths that suit the kernels and not."""
+    for D, M in ((48, 1), (48, 5), (48, 8), (48, 9), (272, 140), (42, 3), (42, 20), (200, 33)):
+        w = ff_weights(cfg, D, dtype)
+        f = ff_module(cfg, w, dtype)
+        g = torch.Generator().manual_seed(M)
+        h = (1.5 * torch.randn((M, D), generator=g)).to(dtype)
+        a, wo = torch.randn((M, 40), generator=g).to(dtype), (torch.randn((D, 40), generator=g) / 40 ** 0.5).to(dtype)
+        want = o.feed_forward(h.double(), {k: v.double() for k, v in w.items()}, "", cfg)
+        assert rel_rms(ff_total(f(h.cuda())), want) < TOL[dtype], (D, M)
+        both = want + a.double() @ wo.double().T
+        assert rel_rms(ff_total(f(h.cuda(), (a.cuda(), wo.cuda()), step=M <= 8)), both) < TOL[dtype], (D, M)
+
+
+def test_the_clamp_acts_on_both_sides(dec):
+    """The gate has an upper limit only; with inputs far beyond the limits the difference shows."""
+    for dtype in DTYPES:
+        cfg = dense(32, 0.5)
+        w = {k: 4 * v for k, v in ff_weights(cfg, 48, dtype).items()}
+        h = (3 * torch.randn((20, 48), generator=torch.Generator().manual_seed(0))).to(dtype)
+        wd = {k: v.double() for k, v in w.items()}
+        want = o.clamped_feed_forward(h.double(), wd, "", 0.5)
+        assert row_errors(o.clamped_feed_forward(h.double(), wd, "", 0.6), want).median() > 0.05
+        f = ff_module(cfg, w, dtype)
+        for rows in (slice(0, 20), slice(0, 8)):
+            assert rel_rms(ff_total(f(h[rows].cuda())), want[rows]) < TOL[dtype]
+
+
+def test_experts_of_very_unequal_load(dec):
+    """All rows to one expert, experts without rows, whole tiles and single rows; the paths agree."""
+    from ternainfer_b200 import decoder_ops as ops
+    D, E, ff, M = 64, 6, 48, 700
+    cfg = moe(E, 2, ff)
+    w = ff_weights(cfg, D, torch.bfloat16)
+    w["router"] *= 0.3
+    h = torch.randn((M, D), generator=torch.Generator().manual_seed(3)).bfloat16()
+    for bias in ([9, 0, 0, 0, 0, 0], [0, 9, 0, 0, 20, 0], [1, 0, -1, 2, 0, -30]):
+        w["router.b"] = torch.tensor(bias).bfloat16()
+        f = ff_module(cfg, w, torch.bfloat16)
+        want = o.experts(h.double(), {k: v.double() for k, v in w.items()}, "", cfg)
+        got = ff_total(f(h.cuda()))
+        assert rel_rms(got, want) < TOL[torch.bfloat16]
+        out, slots, weight = ops.expert_rows(h.cuda(), f.router, f.router_bias, 2, f.up, f.down, f.gate, plain=True)
+        assert rel_rms((out.double()[slots.long()] * weight.double()[..., None]).sum(1), want) < TOL[torch.bfloat16]
+        assert rel_rms(torch.cat([ff_total(f(h[i:i + 7].cuda())) for i in range(0, 70, 7)]), want[:70]) < TOL[torch.bfloat16]
+
+
+@pytest.mark.parametrize("rows,G,N,K", [(300, 1, 512, 192), (129, 1, 16, 8), (1000, 3, 272, 200), (70, 5, 48, 1000), (5000, 2, 1040, 64), (64, 1, 256, 64)])
+def test_grouped_gemm(dec, rows, G, N, K):
+    from ternainfer_b200 import decoder_ops as ops
+    g = torch.Generator().manual_seed(0)
+    x, w = torch.randn((rows, K), generator=g).bfloat16(), (torch.randn((G, N, K), generator=g) / K ** 0.5).bfloat16()
+    bias = torch.randn((G, N), generator=g)
+    split = torch.sort(torch.randint(0, rows + 1, (G - 1,), generator=g)).values.tolist()
+    edges = [0] + split + [rows]
+    counts = None if G == 1 else torch.tensor([b - a for a, b in zip(edges, edges[1:])], dtype=torch.int32, device="cuda")
+    want = torch.cat([x[a:b].double() @ w[i].double().T + bias[i].double() for i, (a, b) in enumerate(zip(edges, edges[1:]))])
+    assert rel_rms(ops.group_gemm(x.cuda(), w.cuda(), counts, bias.cuda()), want) < 5e-3
+    z = want.view(rows, N // 16, 2, 8)
+    for gate, fn in ((ops.silu_gate(), lambda a, b: o.silu(a) * b),
+                     (ops.clamped_gate(1.3, 0.9), lambda a, b: a.clamp(max=0.9) * torch.sigmoid(1.3 * a.clamp(max=0.9)) * (b.clamp(-0.9, 0.9) + 1))):
+        got = ops.group_gemm(x.cuda(), w.cuda(), counts, bias.cuda(), gate)
+        assert rel_rms(got, fn(z[:, :, 0], z[:, :, 1]).reshape(rows, N // 2)) < 6e-3
+
+
+@pytest.mark.parametrize("M", [1, 8])
+def test_linear_with_an_input_per_segment(dec, M):
+    from ternainfer_b200 import decoder_ops as ops
+    g = torch.Generator().manual_seed(0)
+    x, w = torch.randn((5, M, 200), generator=g).bfloat16(), (torch.randn((4 * 48 + 24, 200), generator=g) / 14).bfloat16()
+    got = ops.rows_linear(x.cuda(), w.cuda(), seg_rows=48)
+    want = torch.cat([x[i].double() @ w[48 * i:48 * (i + 1) if i < 4 else None].double().T for i in range(5)], 1)
+    assert rel_rms(got, want) < 5e-3
+
+
+def test_bad_calls_are_refused_on_the_host(dec):
+    from ternainfer_b200 import decoder_ops as ops
+    from ternainfer_b200.lib import DecoderOpsError, GroupGemmArgs, LatentAttnArgs, MoeArgs, WkvArgs
+    ref = ctypes.byref
+    assert dec.decoder_wkv(ref(WkvArgs(B=1, T=1, H=1, dk=300, dv=300, rank=1)), 0, 0, None) == 1
+    assert dec.decoder_wkv(ref(WkvArgs(B=1, T=40, H=1, dk=8, dv=8, rank=1, n_seg=2, seg_len=16)), 0, 0, None) == 1
+    assert dec.decoder_wkv(ref(WkvArgs(B=1, T=1, H=1, dk=8, dv=8, rank=1)), 0, 0, None) == 2
+    assert dec.decoder_latent_step(ref(LatentAttnArgs(B=1, T=1, H=1, R=8, ld=16, slots=4, vdim=8, splits=1)), 0, None) == 2
+    assert dec.decoder_group_gemm(ref(GroupGemmArgs(rows=4, groups=1, N=8, K=8)), None) == 1
+    assert dec.decoder_moe_route(ref(MoeArgs(M=1, E=4, top=5, K=8, ff=8)), 0, None) == 1
+    with pytest.raises(DecoderOpsError):
+        x = torch.zeros((1, 2, 16), device="cuda")          # two streams
+        ops.hyper_norm(x, torch.zeros(16, device="cuda"), 1e-5, torch.float32, y=torch.zeros((1, 16), device="cuda"), y2=torch.zeros((1, 16), device="cuda"))
+    with pytest.raises(TypeError):
+        ops.group_gemm(torch.zeros((16, 16), device="cuda"), torch.zeros((1, 16, 16), device="cuda"))
+
+
+# ------------------------------------------------------------------------------- the model
+
+def make_model(cfg, dtype, max_len, seed=0, rank=6, dic=None):
+    from ternainfer_b200.sidirax import Sidirax, parse_config
+    dic = dic or weights(cfg, seed, rank)
+    return Sidirax(parse_config(cfg), dic, max_seq_len=max_len, dtype=dtype).cuda(), dic
+
+
+def run_engine(model, toks, parts, engine=None, name="r"):
+    from ternainfer_b200.generate import StepEngine
+    e = engine or StepEngine(model)
+    got = torch.cat([e.step(name, toks[a:b], list(range(b - a))) for a, b in parts])
+    e.finish(name)
+    return got
+
+
+MODEL_TOL = {torch.float32: 1e-4, torch.bfloat16: 6e-2}
+
+
+def close(got, want, dtype, cfg):
+    """Every row; but in bf16 rounding may turn a close choice of experts round, and what follows in the sequence with it."""
+    e, tol = row_errors(got, want), MODEL_TOL[dtype]
+    if dtype == torch.float32 or not any(layer["mlp"] and layer["mlp"]["kind"] == "moe" for layer in cfg["layers"]):
+        return e.max() < tol
+    return (e > tol).double().mean() <= 0.3 and e.median() < 0.6 * tol
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", list(CONFIGS))
+def test_model_whole_portions_and_decoding(dec, name, dtype):
+    cfg = CONFIGS[name]
+    T = 110
+    model, dic = make_model(cfg, dtype, T)
+    toks = tokens(cfg, T)
+    want, _ = o.forward(cfg, dic, toks)
+    for parts in ([(0, T)], cuts(T, [25, 2, 40, 3]), cuts(T, [2]), [(0, 60)] + singles(60, T), singles(0, T), cuts(T, [9])):
+        got = run_engine(model, toks, parts)
+        assert close(got, want, dtype, cfg), (parts[:3], row_errors(got, want).topk(5))
+
+
+@pytest.mark.parametrize("name", list(CONFIGS))
+def test_model_layer_by_layer(dec, name):
+    cfg = CONFIGS[name]
+    model, dic = make_model(cfg, torch.float32, 40)
+    toks = tokens(cfg, 40)
+    _, after = o.forward(cfg, dic, toks)
+    seen = {}
+    with torch.inference_mode():
+        model(torch.tensor([toks], device="cuda"), model.make_cache(1, "cuda"), pos(0, 40), start=0, on_layer=seen.__setitem__)
+    assert sorted(seen) == list(range(len(cfg["layers"])))
+    for i, x in seen.items():
+        assert rel_rms(x, after[i]) < 2e-5
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", ["mixed", "no_experts"])
+def test_batches_of_sequences(dec, name, dtype):
+    """Equal-length sequences of one forward against each alone, in prompts and decoding, batches below and above the decode
+    kernels' eight rows."""
+    cfg = CONFIGS[name]
+    T = 50
+    model, dic = make_model(cfg, dtype, T)
+    for B in (3, 11):
+        toks = [tokens(cfg, T, seed=s) for s in range(B)]
+        cache, got = model.make_cache(B, "cuda"), []
+        with torch.inference_mode():
+            for a, b in [(0, 30), (30, 32)] + singles(32, T):
+                got.append(model(torch.tensor([t[a:b] for t in toks], device="cuda"), cache, pos(a, b), start=a))
+        got = torch.cat(got, 1)
+        for i in range(0, B, 2):
+            assert close(got[i], o.forward(cfg, dic, toks[i])[0], dtype, cfg), (B, i, row_errors(got[i], o.forward(cfg, dic, toks[i])[0]))
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_requests_side_by_side_and_caches_used_again(dec, dtype):
+    """Unequal requests interleaved step by step, some finished early and their caches taken over, each against itself alone."""
+    from ternainfer_b200.generate import StepEngine
+    cfg = CONFIGS["mixed"]
+    model, dic = make_model(cfg, dtype, 90)
+    req = {n: tokens(cfg, t, seed=i) for i, (n, t) in enumerate([("a", 90), ("b", 1), ("c", 47), ("d", 61), ("e", 20)])}
+    alone = {n: run_engine(model, t, cuts(len(t), [11, 1, 2])) for n, t in req.items()}
+    e = StepEngine(model)
+    got = {n: [] for n in req}
+    queue, live, at = list(req), [], {n: 0 for n in req}
+    while queue or live:
+        while queue and len(live) < 3:
+            live.append(queue.pop(0))
+        for n in list(live):
+            size = [11, 1, 2][len(got[n]) % 3]
+            t = req[n][at[n]:at[n] + size]
+            got[n].append(e.step(n, t, list(range(len(t)))))
+            at[n] += len(t)
+            if at[n] == len(req[n]):
+                e.finish(n)
+                live.remove(n)
+    assert e.pool.made == 3
+    for n in req:
+        assert torch.equal(torch.cat(got[n]), alone[n]), n
+        assert close(alone[n], o.forward(cfg, dic, req[n])[0], dtype, cfg)
+
+
+def test_wanted_places_and_bad_tokens(dec):
+    from ternainfer_b200.generate import StepEngine
+    cfg = CONFIGS["odd"]
+    model, _ = make_model(cfg, torch.float32, 30)
+    toks = tokens(cfg, 20)
+    e = StepEngine(model)
+    every = e.step("a", toks, list(range(20)))
+    some = e.step("b", toks, [13, 0, 19])
+    assert rel_rms(some, every[[13, 0, 19]]) < 1e-5
+    with pytest.raises(ValueError):
+        e.step("c", [cfg["vocab"]], [])
+
+
+def test_long_decoding(dec):
+    layers = [latent(4, 32, 16, 32, 24, 48, 0.25, dense(64, 1.0)), wkv(2, 32, None), latent(2, 16, 16, 16, 16, 48, 0.3, moe(4, 2, 16), kv_from=0)]
+    for dtype in DTYPES:
+        cfg = config(layers[:2 if dtype == torch.bfloat16 else 3], vocab=61, width=40)
+        model, dic = make_model(cfg, dtype, 420)
+        toks = tokens(cfg, 420)
+        want, _ = o.forward(cfg, dic, toks)
+        got = run_engine(model, toks, [(0, 5)] + singles(5, 420))
+        assert close(got, want, dtype, cfg) and close(got[-40:], want[-40:], dtype, cfg)
+
+
+def test_a_shared_latent_is_the_other_layers(dec):
+    """Changing the latent projection of the layer that owns the cache changes the layer that reads it, also with the
+    owner's own attention silenced."""
+    cfg = config([latent(2, 16, 16, 16, 16, 24, 0.3, None), latent(3, 16, 16, 32, 24, 24, 0.3, None, kv_from=0)], width=40)
+    dic = weights(cfg)
+    dic["l0.mix.o"] = torch.zeros_like(dic["l0.mix.o"])
+    toks = tokens(cfg, 60)
+    other = dict(dic, **{"l0.mix.dkv": dic["l0.mix.dkv"].flip(0)})
+    assert rel_rms(o.forward(cfg, other, toks)[0], o.forward(cfg, dic, toks)[0]) > 0.05
+    for d in (dic, other):
+        for dtype in DTYPES:
+            model, _ = make_model(cfg, dtype, 60, dic=d)
+            for parts in ([(0, 60)], cuts(60, [20, 2]), [(0, 30)] + singles(30, 60)):
+                assert close(run_engine(model, toks, parts), o.forward(cfg, d, toks)[0], dtype, cfg)
+
+
+@pytest.mark.parametrize("graph", [True, False])
+@pytest.mark.parametrize("name", ["mixed", "recurrent_only"])
+def test_greedy_generation_through_fastgen(dec, name, graph):
+    """The generation loop in fp32 chooses the restatement's tokens, for two prompts in one batch; twice in a row
+    from the same caches."""
+    from ternainfer_b200.generate import FastGen, GenArgs
+    cfg = CONFIGS[name]
+    P, N = 23, 30
+    model, dic = make_model(cfg, torch.float32, P + N)
+    prompts = [tokens(cfg, P, seed=s) for s in (3, 4)]
+    gen = FastGen(model, GenArgs(N, 2, P, graph))
+    for turn in range(2):
+        out, _ = gen.generate(torch.tensor(prompts if turn == 0 else prompts[::-1], device="cuda"))
+        for b, p in enumerate(prompts if turn == 0 else prompts[::-1]):
+            seq = p + out[b].tolist()
+            want, _ = o.forward(cfg, dic, seq[:-1])
+            for i in range(N):
+                row = want[P - 1 + i]
+                assert row.max() - row[seq[P + i]] < 1e-4 * row.abs().max(), (turn, b, i)
+
+
+def test_greedy_generation_bf16_follows_its_own_logits(dec):
+    from ternainfer_b200.generate import FastGen, GenArgs
+    cfg = CONFIGS["wide"]
+    model, dic = make_model(cfg, torch.bfloat16, 60)
+    prompt = tokens(cfg, 33, seed=9)
+    out, stats = FastGen(model, GenArgs(27, 1, 33, True)).generate(torch.tensor([prompt], device="cuda"))
+    seq = prompt + out[0].tolist()
+    got = run_engine(model, seq[:-1], [(0, 33)] + singles(33, 59))
+    for i in range(27):
+        row = got[32 + i]
+        assert row.max() - row[seq[33 + i]] < 3e-2 * row.abs().max()
+    assert stats["decode_tokens_per_s"] > 0
+
+
+@pytest.mark.parametrize("dtype", ["bfloat16", "float32"])
+def test_trace_run_program(dec, tmp_path, dtype):
+    cfg = CONFIGS["mixed"]
+    dic = weights(cfg)
+    save_model(tmp_path, cfg, dic)
+    (tmp_path / "out").mkdir()
+    a, b = tokens(cfg, 40, 1), tokens(cfg, 9, 2)
+    steps = [{"step": 0, "entries": [{"id": "x", "tokens": a[:30], "want": list(range(30))}], "end": []},
+             {"step": 1, "entries": [{"id": "x", "tokens": a[30:31], "want": [0]}], "end": []},
+             {"step": 2, "entries": [{"id": "x", "tokens": a[31:], "want": []}], "end": ["x"]},
+             {"step": 3, "entries": [{"id": "y", "tokens": b, "want": list(range(9))}], "end": ["y"]}]
+    p = subprocess.run([os.path.join(ROOT, "bin", "trace_run"), "--model", str(tmp_path), "--dtype", dtype, "--out", str(tmp_path / "out"),
+                        "--max-tokens", "40"], input="\n".join(map(json.dumps, steps)) + "\n", capture_output=True, text=True, timeout=300)
+    assert p.returncode == 0, p.stderr[-2000:]
+    assert [l for l in p.stdout.split("\n") if l.startswith("done")] == [f"done {i}" for i in range(4)]
+    assert sorted(os.listdir(tmp_path / "out")) == ["0.f32", "1.f32", "3.f32"]
+    wa, wb = o.forward(cfg, dic, a)[0], o.forward(cfg, dic, b)[0]
+    got = [torch.from_numpy(np.fromfile(tmp_path / "out" / f"{f}.f32", "<f4").reshape(-1, cfg["vocab"])) for f in (0, 1, 3)]
+    assert close(torch.cat(got), torch.cat([wa[:31], wb]), getattr(torch, dtype), cfg)
+
+
+def test_generate_command_line(dec, tmp_path):
+    cfg = CONFIGS["recurrent_only"]
+    save_model(tmp_path, cfg, weights(cfg))
+    p = subprocess.run([sys.executable, "-m", "ternainfer_b200.generate", "--model", str(tmp_path), "--prompt", "5,9,60,2", "--gen_length", "6"],
+                       capture_output=True, text=True, timeout=300, cwd=ROOT)
+    assert p.returncode == 0, p.stderr[-2000:]
+    assert len(json.loads(p.stdout[p.stdout.index("tokens [") + 7:])) == 6
