@@ -1118,6 +1118,31 @@ def model_speed(torch, build, size, args):
     return out
 
 
+def kernel_table(torch, out, args):
+    """put(model, name, calls, bytes, flops): times the calls and files microseconds, algorithmic bytes and matrix FLOPs, and
+    the fraction of the larger of the two bounds under out[model][name]."""
+    peak, tf = out["peaks"]["hbm_gbs"], out["peaks"]["bf16_tflops"]
+
+    def put(model, name, calls, nbytes, flops=0.0):
+        us = graph_us(torch, calls, max(5, args.steps // 5), args.warmup)
+        bound = max(nbytes / peak / 1e3, flops / tf / 1e6)
+        out[model][name] = {"us": us, "bytes": nbytes, "flops": flops, "bound_us": bound, "frac": bound / us}
+        torch.cuda.empty_cache()
+    return put
+
+
+def copies(nbytes):
+    """Copies of an operand that together are larger than the L2."""
+    return max(2, min(400, int(160e6 / nbytes) + 1))
+
+
+def measured_tflops():
+    try:
+        return float(json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json")))["bf16_tflops"])
+    except Exception:
+        return 1590.0
+
+
 def kepovik_kernels(torch, size, args):
     """Every kernel of both models at this size: microseconds, algorithmic bytes and matrix FLOPs, and the fraction of the
     larger of the two bounds (measured copy rate, measured bf16 GEMM rate; the int8 GEMM against the latter too)."""
@@ -1125,24 +1150,12 @@ def kepovik_kernels(torch, size, args):
     from ternainfer_b200.linear import lm_head_argmax, rmsnorm_quant
     width, ff, heads, kv, dim, dh, dd, _ = KEPOVIK_SIZES[size]
     peak, kind = measured_peak()
-    try:
-        tf = float(json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json")))["bf16_tflops"])
-    except Exception:
-        tf = 1590.0
+    tf = measured_tflops()
     S, V, bf, dev = KEPOVIK_STREAMS, KEPOVIK_VOCAB, torch.bfloat16, "cuda"
     g = torch.Generator(device=dev).manual_seed(args.seed)
     rnd = lambda *shape, dtype=bf, scale=1.0: (scale * torch.randn(shape, generator=g, device=dev)).to(dtype)
     out = {"peaks": {"hbm_gbs": peak, "bf16_tflops": tf, "kind": kind}, "kepovik": {}, "ternary": {}}
-    full = 160e6                                       # more than the L2
-
-    def put(model, name, calls, nbytes, flops=0.0):
-        us = graph_us(torch, calls, max(5, args.steps // 5), args.warmup)
-        bound = max(nbytes / peak / 1e3, flops / tf / 1e6)
-        out[model][name] = {"us": us, "bytes": nbytes, "flops": flops, "bound_us": bound, "frac": bound / us}
-        torch.cuda.empty_cache()
-
-    def copies(nbytes):
-        return max(2, min(400, int(full / nbytes) + 1))
+    put = kernel_table(torch, out, args)
 
     nd, na = 5 * dh * dd + KEPOVIK_RANK, 2 * heads * dim + 2 * kv * dim
     off_d = {n: i * dh * dd for i, n in enumerate(("r", "k", "v", "a", "g", "w1"))}
@@ -1251,6 +1264,182 @@ def run_kepovik_arm(args):
     print(json.dumps(line), flush=True)
 
 
+# ----------------------------------------------------------------------------
+# Sidirax workload: the decoder of ternainfer_b200/sidirax.py beside Kepovik of equal
+# width, layers, heads and active feed-forward width (the closest model: recurrent and
+# attention layers with dense bf16 weights), whole models and kernel by kernel.
+# ----------------------------------------------------------------------------
+
+SIDIRAX_EXPERTS, SIDIRAX_TOP, SIDIRAX_ROT, SIDIRAX_KV_RANK = 32, 4, 64, 512
+
+
+def sidirax_config(size):
+    """wkv and latent attention layers in turn, every second attention layer on the latent of the one before; the first
+    feed-forward dense, the others experts whose chosen ones together are as wide."""
+    width, ff, heads, _, dim, wh, wd, layers = KEPOVIK_SIZES[size]
+    rot = {"base": 10000.0, "dims": SIDIRAX_ROT, "scaling": {"factor": 4.0, "original": 1024, "fast": 32.0, "slow": 1.0}}
+    out = []
+    for i in range(layers):
+        mlp = {"kind": "dense", "ff": ff, "limit": 7.0} if i == 0 else \
+            {"kind": "moe", "expert": {"ff": ff // SIDIRAX_TOP}, "router": {"experts": SIDIRAX_EXPERTS, "top": SIDIRAX_TOP}}
+        if i % 2 == 0:
+            out.append({"type": "wkv", "mixer": {"heads": wh, "dim": wd}, "mlp": mlp})
+            continue
+        mixer = {"heads": heads, "dim": dim, "rot_dim": SIDIRAX_ROT, "vdim": dim, "q_rank": width // 2, "kv_rank": SIDIRAX_KV_RANK,
+                 "scale": (dim + SIDIRAX_ROT) ** -0.5, "rot": rot}
+        if i % 4 == 3:
+            mixer["kv_from"] = i - 2
+        out.append({"type": "latent_attention", "mixer": mixer, "mlp": mlp})
+    return {"architecture": "Sidirax", "vocab": KEPOVIK_VOCAB, "width": width, "norm": {"eps": 1e-5}, "layers": out}
+
+
+def sidirax_model(size, max_len, seed):
+    import torch
+    from ternainfer_b200.sidirax import Sidirax, parse_config, random_checkpoint
+    args = parse_config(sidirax_config(size))
+    return Sidirax(args, random_checkpoint(args, KEPOVIK_RANK, seed), max_seq_len=max_len, dtype=torch.bfloat16).cuda()
+
+
+def sidirax_kernels(torch, size, args):
+    """Every kernel of the model at this size; bytes count every weight that is used once (for experts: the distinct chosen
+    ones), every cache entry and every activation once."""
+    from ternainfer_b200 import decoder_ops as ops
+    width, ff, heads, _, dim, wh, wd, _ = KEPOVIK_SIZES[size]
+    peak, kind = measured_peak()
+    out = {"peaks": {"hbm_gbs": peak, "bf16_tflops": measured_tflops(), "kind": kind}, "sidirax": {}}
+    table = kernel_table(torch, out, args)
+    put = lambda name, calls, nbytes, flops=0.0: table("sidirax", name, calls, nbytes, flops)
+    bf, dev, eps = torch.bfloat16, "cuda", 1e-5
+    g = torch.Generator(device=dev).manual_seed(args.seed)
+    rnd = lambda *shape, dtype=bf, scale=1.0: (scale * torch.randn(shape, generator=g, device=dev)).to(dtype)
+    f32 = lambda *shape, scale=0.3: rnd(*shape, dtype=torch.float32, scale=scale)
+    E, top, rot, R, V, n = SIDIRAX_EXPERTS, SIDIRAX_TOP, SIDIRAX_ROT, SIDIRAX_KV_RANK, KEPOVIK_VOCAB, wh * wd
+    fe, qr, dq, ld, rank, S = ff // top, width // 2, dim + rot, R + rot, KEPOVIK_RANK, 2048
+    trig, w1, mu, silu = f32(S, rot), f32(width), f32(5, width), ops.silu_gate()
+    clamp = ops.clamped_gate(1.702, 7.0)
+    uk, uv, sink = rnd(heads * dim, R, scale=R ** -0.5), rnd(heads * dim, R, scale=R ** -0.5), f32(heads)
+    uk_t = uk.view(heads, dim, R).transpose(1, 2).contiguous()
+    w2, w0, u, nw = rnd(n, rank, scale=0.1), f32(n) - 3, f32(wh, wd), f32(n)
+    rw, rb = rnd(E, width, scale=width ** -0.5), f32(E)
+    up = [rnd(E, 2 * fe, width, scale=width ** -0.5) for _ in range(2)]
+    down = [rnd(E, width, fe, scale=fe ** -0.5) for _ in range(2)]
+    wo = [rnd(width, n, scale=n ** -0.5) for _ in range(8)]
+    for B in (1, 8):
+        tag, at = f"decode_batch{B}", torch.tensor([S - 1], device=dev)
+        for name, N, K in (("latent_in", qr + R + rot, width), ("latent_uq", heads * dq, qr)):
+            nb = 2.0 * (N * K + B * (N + K))
+            x, ws = rnd(B, K), [rnd(N, K, scale=K ** -0.5) for _ in range(copies(nb))]
+            put(f"{tag}/linear_{name}", [lambda w=w: ops.linear(x, w, step=True) for w in ws], nb, 2.0 * B * N * K)
+        N = 4 * n + rank
+        nb = 2.0 * (N * width + B * (N + 5 * width))
+        x, ws = rnd(5, B, width), [rnd(N, width, scale=width ** -0.5) for _ in range(copies(nb))]
+        put(f"{tag}/linear_wkv_in", [lambda w=w: ops.rows_linear(x, w, seg_rows=n, step=True) for w in ws], nb, 2.0 * B * N * width)
+        nb = 2.0 * (2 * ff * width + B * (ff + width))
+        x, ws, bias = rnd(B, width), [rnd(2 * ff, width, scale=width ** -0.5) for _ in range(copies(nb))], f32(2 * ff)
+        put(f"{tag}/dense_up_clamped", [lambda w=w: ops.rows_linear(x, w, bias, clamp, step=True) for w in ws], nb, 4.0 * B * ff * width)
+        nb = 2.0 * (ff * width + width * n + B * (ff + n + width))
+        act, a, ws, db = rnd(B, ff), rnd(B, n), [rnd(width, ff, scale=ff ** -0.5) for _ in range(copies(nb))], f32(width)
+        put(f"{tag}/dense_down_and_mixer_out", [lambda w=w, o=wo[i % 8]: ops.down_step(act, w, db, rest=a, w_rest=o, step=True) for i, w in enumerate(ws)],
+            nb, 2.0 * B * (ff + n) * width)
+        del ws
+        xs = [rnd(B, width) for _ in range(20)]
+        used, acts = [], []
+        for x in xs:
+            acts.append(ops.expert_step(x, rw, rb, top, up[0], silu))
+            used.append(acts[-1][1].unique().numel())
+        used = sum(used) / len(used)
+        put(f"{tag}/router_and_expert_up", [lambda x=x, w=up[i % 2]: ops.expert_step(x, rw, rb, top, w, silu, True) for i, x in enumerate(xs)],
+            2.0 * (used * 2 * fe * width + E * width + B * (width + top * fe)), 4.0 * B * top * fe * width)
+        put(f"{tag}/expert_down_and_mixer_out", [lambda t=t, w=down[i % 2], o=wo[i % 8]: ops.down_step(t[0], w, None, t[1], t[2], a, o, True)
+                                                 for i, t in enumerate(acts)],
+            2.0 * (used * fe * width + width * n + B * (top * fe + n + width)), 2.0 * B * (top * fe + n) * width)
+        xr, y, prev = f32(B, 1, width), rnd(B, width), rnd(B, width)
+        put(f"{tag}/residual_norm", [lambda: ops.hyper_norm(xr, w1, eps, bf, y=y, step=True)] * 20, 12.0 * B * width)
+        put(f"{tag}/residual_norm_shift", [lambda: ops.hyper_norm(xr, w1, eps, bf, y=y, shift=(mu, prev, at), step=True)] * 20, B * width * 26.0 + 20.0 * width)
+        nb = B * wh * wd * wd * 8.0 + 2.0 * n * rank + 12.0 * B * n
+        st, z = [torch.zeros((B, wh, wd, wd), device=dev) for _ in range(copies(nb))], rnd(B, 4 * n + rank)
+        r, k, v, gt, t1 = (z[:, i * n:] for i in range(5))
+        put(f"{tag}/wkv_step", [lambda s=s: ops.wkv(r, k, v, gt, t1, w2, w0, u, nw, s, at, 1, eps, True) for s in st], nb)
+        del st
+        nb = 2.0 * B * S * ld + 4.0 * heads * dim * R
+        cc = [rnd(B, S, ld) for _ in range(copies(2.0 * B * S * ld))]
+        z, q, qn, kn = rnd(B, qr + ld), rnd(B, heads * dq), f32(qr), f32(R)
+        qa = ops.absorb(q, uk, uk_t, heads, dim, rot, R, ld, trig, at, 1)
+        put(f"{tag}/latent_norms_append", [lambda c=c: ops.latent_prep(z, 0, qn, at, 1, eps, c, qr, kn, R, rot, trig, True) for c in cc], 4.0 * B * (qr + ld))
+        put(f"{tag}/latent_absorb", [lambda: ops.absorb(q, uk, uk_t, heads, dim, rot, R, ld, trig, at, 1, True)] * 20, 2.0 * (heads * dim * R + B * heads * (dq + ld)))
+        put(f"{tag}/latent_attention_2048", [lambda c=c: ops.latent_attention_step(qa, c, uv, sink, at, 1, dim, 0.07, True) for c in cc],
+            2.0 * B * S * ld + 2.0 * heads * dim * R, 2.0 * B * heads * S * (ld + R))
+        put(f"{tag}/latent_attention_2048_all", [lambda c=c: ops.latent_attention_step(ops.absorb(q, uk, uk_t, heads, dim, rot, R, ld, trig, at, 1, True), c, uv, sink,
+                                                                                       at, 1, dim, 0.07, True) for c in cc], nb, 2.0 * B * heads * S * (ld + R))
+        del cc
+        hd, W = rnd(B, width), rnd(V, width, scale=width ** -0.5)
+        put(f"{tag}/output_head", [lambda: ops.output_argmax(hd, W)], 2.0 * V * width)
+        del W
+    T, tag = S, "prefill2048"
+    pos, h = torch.arange(T, device=dev), rnd(T, width)
+    xr, y, ye = [f32(T, 1, width) for _ in range(4)], rnd(T, width), rnd(T * top, width)
+    slots, sw = torch.randperm(T * top, device=dev).int().view(T, top), torch.rand((T, top), device=dev)
+    put(f"{tag}/residual_norm", [lambda x=x: ops.hyper_norm(x, w1, eps, bf, y=y) for x in xr], T * width * 12.0)
+    put(f"{tag}/residual_norm_experts", [lambda x=x: ops.hyper_norm(x, w1, eps, bf, y=y, y2=ye, slots=slots, slot_w=sw) for x in xr], T * width * (12.0 + 2 * top))
+    del xr, ye
+    prev = rnd(1, width)
+    put(f"{tag}/token_shift", [lambda: ops.token_shift(h, mu, prev, pos, T)] * 5, T * width * 12.0)
+    zs, state = [rnd(4, T, n) for _ in range(2)], torch.zeros((1, wh, wd, wd), device=dev)
+    t1, zw = rnd(T, rank), f32(T, n)
+    put(f"{tag}/wkv", [lambda z=z: ops.wkv(z[0], z[1], z[2], z[3], t1, w2, w0, u, nw, state, pos, T, eps, zw=zw) for z in zs], T * n * 14.0)
+    out["sidirax"][f"{tag}/wkv"]["fp32_fma"] = 2.0 * T * n * wd
+    x5, ws = rnd(4, T, width), [rnd(4, n, width, scale=width ** -0.5) for _ in range(4)]
+    put(f"{tag}/linear_wkv_in", [lambda w=w: torch.bmm(x5, w.transpose(1, 2)) for w in ws], 8.0 * (T * (n + width) + n * width), 8.0 * T * n * width)
+    del zs, ws, x5
+    cache, ukv = rnd(1, T, ld), torch.cat([uk, uv])
+    qs = [rnd(T, heads * dq) for _ in range(5)]
+    att = T * (T + 1.0) * heads * (dq + dim)
+    put(f"{tag}/attention", [lambda q=q: ops.latent_attention_prompt(q, ukv, cache, sink, 0, T, heads, dim, rot, dim, R, 0.07) for q in qs],
+        2.0 * T * (heads * (dq + dim) + ld), att + 4.0 * T * R * heads * dim)
+    put(f"{tag}/expand_keys_values", [lambda: torch.mm(cache[0, :, :R], ukv.t())] * 5, 2.0 * T * (R + 2 * heads * dim), 4.0 * T * R * heads * dim)
+    put(f"{tag}/rotate_queries", [lambda q=q: ops.rotate(q, q, heads, dim, dim, rot, trig, pos, T) for q in qs], 4.0 * T * heads * rot)
+    z, qn, kn = rnd(T, qr + ld), f32(qr), f32(R)
+    put(f"{tag}/latent_norms_append", [lambda: ops.latent_prep(z, 0, qn, pos, T, eps, cache, qr, kn, R, rot, trig)] * 5, 4.0 * T * (qr + ld))
+    del qs
+    ws, bias = [rnd(2 * ff, width, scale=width ** -0.5) for _ in range(3)], f32(2 * ff)
+    nb, fl = 2.0 * (T * (width + ff) + 2 * ff * width), 4.0 * T * ff * width
+    put(f"{tag}/dense_up_clamped", [lambda w=w: ops.gated_linear(h, w, bias, clamp) for w in ws], nb, fl)
+    put(f"{tag}/dense_up_vendor_gemm_alone", [lambda w=w: ops.linear(h, w) for w in ws], nb + 2.0 * T * ff, fl)
+    del ws
+    put(f"{tag}/experts", [lambda i=i: ops.expert_rows(h, rw, rb, top, up[i], down[i], silu) for i in range(2)],
+        2.0 * (3 * E * fe * width + T * width * (1 + top)), 6.0 * T * top * fe * width)
+    rows, counts = rnd(T * top, width), torch.full((E,), T * top // E, dtype=torch.int32, device=dev)
+    put(f"{tag}/expert_up_gemm", [lambda i=i: ops.group_gemm(rows, up[i], counts, gate=silu) for i in range(2)],
+        2.0 * (2 * E * fe * width + T * top * (width + fe)), 4.0 * T * top * fe * width)
+    act = rnd(T * top, fe)
+    put(f"{tag}/expert_down_gemm", [lambda i=i: ops.group_gemm(act, down[i], counts) for i in range(2)],
+        2.0 * (E * fe * width + T * top * (width + fe)), 2.0 * T * top * fe * width)
+    return out
+
+
+def run_sidirax_arm(args):
+    import torch
+    torch.cuda.set_device(0)
+    sampler = ClockSampler(0)
+    sampler.start()
+    res = {}
+    for size in KEPOVIK_SIZES:
+        res[size] = {"layers": KEPOVIK_SIZES[size][-1], "kernels": sidirax_kernels(torch, size, args)}
+        res[size]["kernels"]["kepovik"] = kepovik_kernels(torch, size, args)["kepovik"]
+        if not args.headline_only:
+            res[size].update(sidirax=model_speed(torch, sidirax_model, size, args), kepovik=model_speed(torch, kepovik_model, size, args))
+    clocks = sampler.stop()
+    best = res["2560"].get("sidirax", {}).get("prompt512_batch1", {})
+    line = {"metric": "sidirax_decode_tokens_per_s", "value": best.get("decode_tokens_per_s"), "unit": "tokens/s", "n_gpus": 1,
+            "steps": args.steps, "warmup": args.warmup, "ms_per_step": best.get("decode_ms"), "higher_is_better": True, "scaling": "weak",
+            "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
+            "config": {"workload": "sidirax_2560_30_layers_prompt512_batch1", "vocab": KEPOVIK_VOCAB, "experts": SIDIRAX_EXPERTS, "top": SIDIRAX_TOP,
+                       "kv_rank": SIDIRAX_KV_RANK, "rot_dim": SIDIRAX_ROT, "decay_rank": KEPOVIK_RANK, "seed": args.seed,
+                       "l2_policy": "weights, states and caches larger than L2 in rotation; decode activations stay in L2"},
+            "sizes": res, "clocks": clocks}
+    print(json.dumps(line), flush=True)
+
+
 def _finish(world):
     """Leave without tearing NCCL down: destroying a process group while CUDA
     graphs that hold NCCL kernels are alive blocks at exit, so every rank meets
@@ -1275,13 +1464,13 @@ def main():
     ap.add_argument("--tokens", type=int, default=8)
     ap.add_argument("--layers", type=int, default=30)
     ap.add_argument("--seed", type=int, default=1234)
-    ap.add_argument("--workload", default="sweep", choices=["sweep", "tp", "decode", "list", "head", "prefill", "kepovik"])
+    ap.add_argument("--workload", default="sweep", choices=["sweep", "tp", "decode", "list", "head", "prefill", "kepovik", "sidirax"])
     ap.add_argument("--unfused", action="store_true", help="decode workload: plain torch glue between the linears")
     ap.add_argument("--tp_mode", default="single", choices=["single", "fused", "exact"])
     ap.add_argument("--no_graph", action="store_true", help="tp workload: launch eagerly instead of replaying a CUDA graph")
     ap.add_argument("--verbose", action="store_true")
     ap.add_argument("--headline_only", action="store_true",
-                    help="sweep workload: only the headline and end-to-end legs (short runs for profiling)")
+                    help="sweep workload: only the headline and end-to-end legs (short runs for profiling); sidirax workload: only the kernels")
     args = ap.parse_args()
     args.warmup = max(args.warmup, 3)
     if args.impl == "reference":
@@ -1292,6 +1481,8 @@ def main():
         run_decode_arm(args)
     elif args.workload == "kepovik":
         run_kepovik_arm(args)
+    elif args.workload == "sidirax":
+        run_sidirax_arm(args)
     elif args.workload in ("list", "head", "prefill"):
         run_single_leg(args)
     else:

@@ -227,10 +227,10 @@ typedef struct {
 int decoder_rotate(const decoder_rotate_args* a, int dtype, int pdl, void* stream);
 
 /* Up to eight bf16 rows: queries q [rows][H][dim + rot] (not rotated) to absorbed queries qa [rows][H][ld] in the cache's
- * layout.  R a multiple of 8. */
+ * layout; dim and rot multiples of 8. */
 typedef struct {
     const void* q;
-    const void* w_uk;          /* [H*dim][R] */
+    const void* w_uk_t;        /* [H][R][dim] */
     void* qa;
     const float* trig;         /* [positions][dims] */
     const long long* pos;      /* [T] */
@@ -240,8 +240,8 @@ int decoder_absorb(const decoder_absorb_args* a, int pdl, void* stream);
 
 /* Attention in the absorbed form: causal softmax over the cache with the sink in the denominator.
  * decoder_latent_attn: any type and size, out = weighted latents [rows][H][R].
- * decoder_latent_step: bf16, R a multiple of 8 up to 1024, ld up to decoder_latent_step_width(): the keys in `splits`
- * ranges, then the product with w_uv: y [rows][H*vdim]. */
+ * decoder_latent_step: bf16, R a multiple of 8 up to 1024, ld up to decoder_latent_step_width(): the keys in splits *
+ * cluster ranges, those of a cluster (up to 8) joined on the way, then the product with w_uv: y [rows][H*vdim]. */
 typedef struct {
     const void* qa;            /* [rows][H][ld], rows = B*T */
     const void* cache;         /* [B][slots][ld], ld a multiple of 8 */
@@ -252,7 +252,7 @@ typedef struct {
     float* part;               /* [rows][H][splits][R] */
     float* ml;                 /* [rows][H][splits][2] */
     void* y;                   /* [rows][H*vdim] */
-    int B, T, H, R, ld, vdim, slots, splits;
+    int B, T, H, R, ld, vdim, slots, splits, cluster;
     float scale;
 } decoder_latent_attn_args;
 int decoder_latent_attn(const decoder_latent_attn_args* a, int dtype, int pdl, void* stream);
@@ -277,10 +277,11 @@ int decoder_latent_prompt(const decoder_latent_prompt_args* a, void* stream);
  * decoder_moe_route: chosen experts and weights; with counts (zeroed by the caller) also every choice's rank among its
  *   expert's, then the rows of x sorted by expert, slots[token][j] saying where a choice's row went (bf16, K % 8 = 0).
  * decoder_moe_plain: any type and size, chosen and weight given: act, and out [M*top][D] not weighted.
- * decoder_moe_up_step: bf16, M <= 8: routing and activations in one launch.
+ * decoder_moe_up_step: bf16, M <= 8, K a multiple of 8 up to 12288: routing (router instead of logits) and activations.
  * decoder_moe_down_step: bf16, M <= 8: out [M][D] = weighted sum + w_rest rest + bias.  Dense: weight NULL, E = top = 1. */
 typedef struct {
     const float* logits;       /* [M][E], without bias */
+    const void* router;        /* [E][K] */
     const float* router_bias;  /* [E] */
     int* chosen;               /* [M][top] */
     float* weight;             /* [M][top] */

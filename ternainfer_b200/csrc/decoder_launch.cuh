@@ -33,7 +33,7 @@ inline bool misaligned(const void* p, unsigned n) { return (reinterpret_cast<uin
 
 template <typename... P, typename... Q>
 inline int launch(void (*kernel)(P...), dim3 grid, int threads, size_t smem, int pdl, void* stream, int cluster, Q... args) {
-    if (smem > 48 * 1024 &&
+    if (smem > 16 * 1024 &&   // (what a kernel has beside it in fixed arrays counts towards the 48 KB that need no request)
         cudaFuncSetAttribute(reinterpret_cast<const void*>(kernel), cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
         return bad(DECODER_LAUNCH, "shared memory request refused");
     cudaLaunchConfig_t cfg = {};

@@ -10,12 +10,14 @@
 // Two forms.  Prompts expand keys and values per head (latent_attn_tc.cuh).  Few tokens absorb W_uk into the query
 // and W_uv into the output and read the cache as it is: all heads of a token share one stream of keys, which are
 // their values too.  The kernels here: norms, rotation and cache append; the absorbed form for any type and size;
-// the absorbed form for up to eight bf16 tokens on mma.sync, the keys split over the chip; the join of the parts
-// with the product with W_uv.
+// the absorbed form for few bf16 tokens on mma.sync, the keys split over the chip; the join of the parts with the
+// product with W_uv.
 #pragma once
 #include "decoder_common.cuh"
 #include "decoder_ops.h"
+#include "decoder_status.cuh"
 #include "lm_head.cuh"
+#include "tcgen05_sm100.cuh"
 
 namespace tsp {
 
@@ -28,35 +30,45 @@ typedef decoder_latent_prep_args LatentPrepParams;
 // the cache.  trig [positions][dims] holds cosine and sine of every pair.
 template <typename A>
 __global__ void __launch_bounds__(256) latent_prep_kernel(const LatentPrepParams p) {
-    __shared__ float red[32], red2[32];
+    extern __shared__ __align__(16) float latent_prep_smem[];    // the row's query latent, key latent, key part
+    __shared__ float2 red[8];
     griddep_launch_dependents();
     griddep_wait();
     const int row = blockIdx.x, b = row / p.T, t = row - b * p.T, tid = threadIdx.x;
     const A* z = reinterpret_cast<const A*>(p.z) + (size_t)row * p.ld_z;
-    const A *zq = z + p.off_q, *zk = z + p.off_kv;
+    float *q_s = latent_prep_smem, *k_s = q_s + p.q_rank;
     const long long pos = p.pos[0] + t;
-    float sq = 0.f, sk = 0.f;
+    const bool append = p.cache && pos < p.slots;
+    float2 ss = make_float2(0.f, 0.f);
     for (int c = tid; c < p.q_rank; c += 256) {
-        const float v = ld_cg(zq + c);
-        sq = fmaf(v, v, sq);
+        const float v = ld_cg(z + p.off_q + c);
+        q_s[c] = v;
+        ss.x = fmaf(v, v, ss.x);
     }
-    if (p.cache)
-        for (int c = tid; c < p.R; c += 256) {
-            const float v = ld_cg(zk + c);
-            sk = fmaf(v, v, sk);
+    if (append)
+        for (int c = tid; c < p.R + p.rot; c += 256) {
+            const float v = ld_cg(z + p.off_kv + c);
+            k_s[c] = v;
+            if (c < p.R) ss.y = fmaf(v, v, ss.y);
         }
-    const float iq = 1.f / sqrtf(block_sum(sq, red) / (float)p.q_rank + p.eps);
+    ss = make_float2(warp_sum(ss.x), warp_sum(ss.y));
+    if ((tid & 31) == 0) red[tid >> 5] = ss;
+    __syncthreads();
+    ss = red[0];
+#pragma unroll
+    for (int i = 1; i < 8; ++i) ss.x += red[i].x, ss.y += red[i].y;
+    const float iq = 1.f / sqrtf(ss.x / (float)p.q_rank + p.eps);
     A* cq = reinterpret_cast<A*>(p.cq) + (size_t)row * p.q_rank;
-    for (int c = tid; c < p.q_rank; c += 256) cq[c] = from_f<A>(ld_cg(zq + c) * iq * p.q_norm[c]);
-    if (!p.cache || pos >= p.slots) return;
-    const float ik = 1.f / sqrtf(block_sum(sk, red2) / (float)p.R + p.eps);
+    for (int c = tid; c < p.q_rank; c += 256) cq[c] = from_f<A>(q_s[c] * iq * p.q_norm[c]);
+    if (!append) return;
+    const float ik = 1.f / sqrtf(ss.y / (float)p.R + p.eps);
     A* k = reinterpret_cast<A*>(p.cache) + ((size_t)b * p.slots + pos) * p.ld;
-    for (int c = tid; c < p.R; c += 256) k[c] = from_f<A>(ld_cg(zk + c) * ik * p.kv_norm[c]);
+    for (int c = tid; c < p.R; c += 256) k[c] = from_f<A>(k_s[c] * ik * p.kv_norm[c]);
     const float* trig = p.trig + (size_t)pos * p.dims;
     for (int c = tid; c < p.rot; c += 256) {
-        float v = ld_cg(zk + p.R + c);
+        float v = k_s[p.R + c];
         if (c < p.dims) {
-            const float o = ld_cg(zk + p.R + (c ^ 1)), cs = trig[c & ~1], sn = trig[c | 1];
+            const float o = k_s[p.R + (c ^ 1)], cs = trig[c & ~1], sn = trig[c | 1];
             v = (c & 1) ? v * cs + o * sn : v * cs - o * sn;
         }
         k[p.r_at + c] = from_f<A>(v);
@@ -144,15 +156,15 @@ __global__ void __launch_bounds__(128) latent_attn_plain_kernel(const LatentAttn
 }
 
 // ------------------------------------------------------------------------------------------ few bf16 tokens
-// qa[row][h][r] = sum_d q[row][h][d] W_uk[h][d][r] for up to eight rows, and the rotated part behind it: CTAs
-// x = 128 latents of one head (y), the last x rotates.  Eight warps split d; partial sums meet in shared memory.
+// qa[row][h][r] = sum_d q[row][h][d] W_uk^T[h][r][d] for up to eight rows, and the rotated part behind it: CTAs
+// x = 128 latents of one head (y), 16 per warp as rows of an MMA whose columns are the rows of q; the last x rotates.
+// The weights are requested before the wait.
 typedef decoder_absorb_args AbsorbParams;
 
 static __global__ void __launch_bounds__(256) absorb_kernel(const AbsorbParams p) {
-    extern __shared__ __align__(16) float absorb_smem[];     // q [8][dim], partial sums [8 warps][M][128]
     griddep_launch_dependents();
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.y, dim = p.dim, M = p.B * p.T;
-    const int dq = dim + p.rot;
+    const int dq = dim + p.rot, g = lane >> 2, qd = lane & 3;
     const bf16* q = reinterpret_cast<const bf16*>(p.q);
     bf16* qa = reinterpret_cast<bf16*>(p.qa);
     if (blockIdx.x == gridDim.x - 1) {                       // rotation, and zeros where the layout has gaps
@@ -173,52 +185,35 @@ static __global__ void __launch_bounds__(256) absorb_kernel(const AbsorbParams p
         }
         return;
     }
-    float* q_s = absorb_smem;
-    float* part = q_s + (8 * dim + 3) / 4 * 4;
-    const int r0 = blockIdx.x * 128 + lane * 4;              // R is a multiple of 4: a lane's latents are in or out together
-    const int d0 = dim * warp / 8, d1 = dim * (warp + 1) / 8;
-    const bf16* w = reinterpret_cast<const bf16*>(p.w_uk) + (size_t)h * dim * p.R + r0;
-    const bool in = r0 < p.R;
-    constexpr int PRE = 16;
-    uint2 wv[PRE];
-    auto fetch = [&](int u, int d) { wv[u] = in && d < d1 ? __ldg(reinterpret_cast<const uint2*>(w + (size_t)d * p.R)) : make_uint2(0, 0); };
-#pragma unroll
-    for (int u = 0; u < PRE; ++u) fetch(u, d0 + u);
-    griddep_wait();
-    for (int i = tid; i < M * dim; i += 256) q_s[i] = ld_cg(q + (size_t)(i / dim) * p.H * dq + h * dq + i % dim);
-    __syncthreads();
-    float acc[8][4];
-#pragma unroll
-    for (int m = 0; m < 8; ++m)
-#pragma unroll
-        for (int j = 0; j < 4; ++j) acc[m][j] = 0.f;
-    for (int d = d0; d < d1; d += PRE) {
+    constexpr int PRE = 4;                                   // k-steps of 32 in flight
+    const int r0 = blockIdx.x * 128 + warp * 16;
+    const bool ok0 = r0 + g < p.R, ok1 = r0 + g + 8 < p.R;
+    const bf16* w = reinterpret_cast<const bf16*>(p.w_uk_t) + (size_t)h * p.R * dim + qd * 8;
+    const bf16 *w0 = w + (size_t)(ok0 ? r0 + g : 0) * dim, *w1 = w + (size_t)(ok1 ? r0 + g + 8 : 0) * dim;
+    const bf16* x = q + (size_t)(g < M ? g : 0) * p.H * dq + h * dq + qd * 8;
+    const uint4 zero = make_uint4(0, 0, 0, 0);
+    uint4 a[PRE], b[PRE], xv[PRE];
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+    for (int d = 0; d < dim; d += 32 * PRE) {
 #pragma unroll
         for (int u = 0; u < PRE; ++u) {
-            const float f[4] = {__uint_as_float(wv[u].x << 16), __uint_as_float(wv[u].x & 0xffff0000u), __uint_as_float(wv[u].y << 16),
-                                __uint_as_float(wv[u].y & 0xffff0000u)};
-            if (d + u < d1) {
+            const bool in = d + 32 * u + qd * 8 < dim;
+            a[u] = in && ok0 ? ldg_stream_128(w0 + d + 32 * u) : zero;
+            b[u] = in && ok1 ? ldg_stream_128(w1 + d + 32 * u) : zero;
+        }
+        if (d == 0) griddep_wait();
 #pragma unroll
-                for (int m = 0; m < 8; ++m)
-                    if (m < M) {
-                        const float x = q_s[m * dim + d + u];
+        for (int u = 0; u < PRE; ++u) xv[u] = g < M && d + 32 * u + qd * 8 < dim ? ld_cg_128(x + d + 32 * u) : zero;
 #pragma unroll
-                        for (int j = 0; j < 4; ++j) acc[m][j] = fmaf(f[j], x, acc[m][j]);
-                    }
-            }
-            fetch(u, d + PRE + u);
+        for (int u = 0; u < PRE; ++u) {
+            mma_bf16_16x8x16(acc, a[u].x, b[u].x, a[u].y, b[u].y, xv[u].x, xv[u].y);
+            mma_bf16_16x8x16(acc, a[u].z, b[u].z, a[u].w, b[u].w, xv[u].z, xv[u].w);
         }
     }
 #pragma unroll
-    for (int m = 0; m < 8; ++m)
-        if (m < M) *reinterpret_cast<float4*>(part + ((size_t)warp * M + m) * 128 + lane * 4) = make_float4(acc[m][0], acc[m][1], acc[m][2], acc[m][3]);
-    __syncthreads();
-    for (int i = tid; i < M * 128; i += 256) {
-        const int r = blockIdx.x * 128 + (i & 127);
-        float v = 0.f;
-#pragma unroll
-        for (int k = 0; k < 8; ++k) v += part[k * M * 128 + i];
-        if (r < p.R) qa[((size_t)(i >> 7) * p.H + h) * p.ld + r] = from_f<bf16>(v);
+    for (int c = 0; c < 4; ++c) {
+        const int row = 2 * qd + (c & 1), r = r0 + g + (c >> 1) * 8;
+        if (row < M && r < p.R) qa[((size_t)row * p.H + h) * p.ld + r] = from_f<bf16>(acc[c]);
     }
 }
 
@@ -228,164 +223,242 @@ __device__ __forceinline__ void ldmatrix4(uint32_t addr, uint32_t (&v)[4]) {
 __device__ __forceinline__ void ldmatrix4_trans(uint32_t addr, uint32_t (&v)[4]) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]) : "r"(addr));
 }
-__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, bool in) {   // 16 bytes, zeros when out of range
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(__cvta_generic_to_global(src)), "r"(in ? 16 : 0) : "memory");
+__device__ __forceinline__ float ld_cluster(uint32_t addr, int rank) {
+    float v;
+    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(map_to_rank(addr, rank)));
+    return v;
 }
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N>
-__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+__device__ __forceinline__ float4 ld_cluster4(uint32_t addr, int rank) {
+    float4 v;
+    asm volatile("ld.shared::cluster.v4.f32 {%0,%1,%2,%3}, [%4];" : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w) : "r"(map_to_rank(addr, rank)));
+    return v;
+}
 
-// One CTA: 16 heads of one row against one of gridDim.x ranges of the keys, 64 at a time.  Scores: a warp takes eight
-// keys, k = the latent and rotated columns.  Weighted sum: a warp takes an eighth of the latents.  Output: unnormalised
-// sums, running maximum (base 2) and sum of weights per range.
+// Up to 32 heads of one row against the keys, which are cut into one range per CTA of the grid's x.  Queries and keys, 64
+// at a time, arrive by TMA in boxes of 64 columns with 128-byte swizzle, the next tile under the work on this one.  Scores: a
+// warp takes 16 keys and half of the columns.  Weighted sum: a warp takes an eighth of the latents.  The CTAs of a
+// cluster add their sums up in distributed shared memory, a share of the columns each, and leave unnormalised sums,
+// maximum (base 2) and sum of weights of the cluster's ranges.
 struct LatentStepSmem {
-    int stride, q, s, p, st, kv, total;                      // bytes
-    __host__ __device__ explicit LatentStepSmem(int ld) {
-        stride = ((ld + 15) / 16 * 16 + 8) * 2;              // an odd number of 16-byte units: ldmatrix without conflicts
-        q = 0, s = q + 16 * stride, p = s + 16 * 68 * 4, st = p + 16 * 72 * 2, kv = st + 3 * 16 * 4;
-        kv = (kv + 15) / 16 * 16;
-        total = kv + 2 * 64 * stride;
+    static constexpr int bar = 0, abort_flag = 16, st = 128, data = 1024;    // st: maxima, sums, factors [32] each
+    int boxes, tile, stages, q, s, p, total;                 // bytes, from a 1024-byte boundary
+    __host__ __device__ LatentStepSmem(int ld, int mt, int limit) {
+        boxes = (ld + 63) / 64, tile = boxes * 64 * 128;
+        const int rest = mt * 16 * (boxes * 128 + 2 * 68 * 4 + 72 * 2);
+        stages = 1024 + data + 2 * tile + rest <= limit ? 2 : 1;
+        q = data + stages * tile, s = q + mt * 16 * boxes * 128, p = s + 2 * mt * 16 * 68 * 4;
+        total = 1024 + data + stages * tile + rest;
     }
 };
 
-template <int NT>   // 16-latent tiles per warp: R <= 128 * NT
-__global__ void __launch_bounds__(256) latent_step_kernel(const LatentAttnParams p) {
-    extern __shared__ __align__(16) uint8_t latent_step_smem[];
-    const LatentStepSmem L(p.ld);
-    const uint32_t base = smem_u32(latent_step_smem);
-    float* s_s = reinterpret_cast<float*>(latent_step_smem + L.s);
-    bf16* p_s = reinterpret_cast<bf16*>(latent_step_smem + L.p);
-    float *m_s = reinterpret_cast<float*>(latent_step_smem + L.st), *l_s = m_s + 16, *f_s = m_s + 32;
+template <int NT, int MT>   // 16-latent tiles per warp: R <= 128 * NT; 16-head tiles
+__global__ void __launch_bounds__(256)
+    latent_step_kernel(const LatentAttnParams p, const int smem_limit, const __grid_constant__ CUtensorMap map_q,
+                       const __grid_constant__ CUtensorMap map_cache) {
+    extern __shared__ __align__(128) uint8_t latent_step_smem[];
+    const LatentStepSmem L(p.ld, MT, smem_limit);
+    const uint32_t dyn = smem_u32(latent_step_smem), base = (dyn + 1023u) & ~1023u;
+    uint8_t* mem = latent_step_smem + (base - dyn);
+    volatile int* abort_flag = reinterpret_cast<volatile int*>(mem + L.abort_flag);
+    float *s_s = reinterpret_cast<float*>(mem + L.s), *o_s = reinterpret_cast<float*>(mem + L.data);
+    bf16* p_s = reinterpret_cast<bf16*>(mem + L.p);
+    float *m_s = reinterpret_cast<float*>(mem + L.st), *l_s = m_s + 32, *f_s = m_s + 64;
     griddep_launch_dependents();
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int split = blockIdx.x, splits = gridDim.x, h0 = blockIdx.y * 16, row = blockIdx.z, b = row / p.T, t = row - b * p.T;
-    const int ld = p.ld, words = ld / 8, ksteps = (ld + 15) / 16, hn = min(16, p.H - h0);
+    const int split = blockIdx.x, splits = gridDim.x, C = p.cluster, rank = split % C;
+    const int h0 = blockIdx.y * 16 * MT, row = blockIdx.z, b = row / p.T, t = row - b * p.T;
+    const int ld = p.ld, ksteps = (ld + 15) / 16, hn = min(16 * MT, p.H - h0);
+    if (tid == 0) {
+        mbar_init(base + L.bar, 1), mbar_init(base + L.bar + 8, 1);
+        *abort_flag = 0;
+        mbar_fence_init();
+    }
+    if (tid < 32) m_s[tid] = -INFINITY, l_s[tid] = 0.f;
+    __syncthreads();
     griddep_wait();
     const int n = (int)min(p.pos[0] + t + 1, (long long)p.slots);
     const int lo = (int)((long long)n * split / splits), hi = (int)((long long)n * (split + 1) / splits);
-    const bf16* cache = reinterpret_cast<const bf16*>(p.cache) + (size_t)b * p.slots * ld;
-    const bf16* q = reinterpret_cast<const bf16*>(p.qa) + ((size_t)row * p.H + h0) * ld;
-    auto fetch = [&](int buf, int j0) {                      // every row up to the padded width, zeros outside
-        const int w16 = 2 * ksteps;
-        for (int i = tid; i < 64 * w16; i += 256) {
-            const int r = i / w16, c = i - r * w16;
-            const bool in = j0 + r < hi && c < words;
-            cp_async16(base + L.kv + (buf * 64 + r) * L.stride + c * 16, cache + (in ? (size_t)(j0 + r) * ld + c * 8 : 0), in);
-        }
-        cp_async_commit();
+    const int tiles = (hi - lo + 63) / 64;
+    auto fetch = [&](int it) {                               // one thread; whole 32-row groups, rows beyond hi are masked
+        const int buf = it % L.stages, groups = min(2, (hi - lo - 64 * it + 31) / 32);
+        const uint32_t bar = base + L.bar + 8 * buf;
+        mbar_arrive_expect_tx(bar, groups * L.boxes * 4096 + (it == 0 ? MT * 16 * 128 * L.boxes : 0));
+        if (it == 0)
+            for (int i = 0; i < L.boxes; ++i) tma_load_2d(base + L.q + i * MT * 2048, &map_q, 64 * i, row * p.H + h0, bar);
+        for (int i = 0; i < L.boxes; ++i)
+            for (int r = 0; r < groups; ++r)
+                tma_load_2d(base + L.data + buf * L.tile + i * 8192 + r * 4096, &map_cache, 64 * i, b * p.slots + lo + 64 * it + 32 * r, bar);
     };
-    for (int i = tid; i < 16 * 2 * ksteps; i += 256) {
-        const int r = i / (2 * ksteps), c = i - r * 2 * ksteps;
-        const bool in = r < hn && c < words;
-        cp_async16(base + L.q + r * L.stride + c * 16, q + (in ? (size_t)r * ld + c * 8 : 0), in);
-    }
-    fetch(0, lo);
-    if (tid < 16) m_s[tid] = -INFINITY, l_s[tid] = 0.f;
-    float acc[NT][2][4];
+    if (tid == 0)
+        for (int it = 0; it < min(tiles, L.stages); ++it) fetch(it);
+    float acc[NT][MT][2][4];
 #pragma unroll
     for (int i = 0; i < NT; ++i)
 #pragma unroll
-        for (int j = 0; j < 2; ++j)
+        for (int m = 0; m < MT; ++m)
 #pragma unroll
-            for (int c = 0; c < 4; ++c) acc[i][j][c] = 0.f;
+            for (int j = 0; j < 2; ++j)
+#pragma unroll
+                for (int c = 0; c < 4; ++c) acc[i][m][j][c] = 0.f;
     const int g = lane >> 2, qd = lane & 3;
-    const int tiles = (hi - lo + 63) / 64;
+    const int key0 = (warp & 3) * 16, half = warp >> 2, k0 = half * ((ksteps + 1) / 2), k1 = half ? ksteps : (ksteps + 1) / 2;
+    bool ok = true;
     for (int it = 0; it < tiles; ++it) {
-        const int j0 = lo + it * 64, buf = it & 1;
-        if (it + 1 < tiles) fetch(buf ^ 1, j0 + 64), cp_async_wait<1>();
-        else cp_async_wait<0>();
-        __syncthreads();
-        {   // scores of keys j0 + 8 warp .. + 7
-            float d0[4] = {0.f, 0.f, 0.f, 0.f}, d1[4] = {0.f, 0.f, 0.f, 0.f};
-            const uint32_t qa = base + L.q + (lane & 15) * L.stride + (lane >> 4) * 16;
-            const uint32_t ka = base + L.kv + (buf * 64 + warp * 8 + (lane & 7)) * L.stride + (lane >> 3) * 16;
-            for (int k = 0; k < ksteps; k += 2) {
-                uint32_t a[4], a2[4], kb[4];
-                ldmatrix4(qa + k * 32, a);
-                // four 8-column pieces of the keys: two k-steps (the second may lie in the row's padding, read but unused)
-                if (k + 1 < ksteps) {
-                    ldmatrix4(ka + k * 32, kb);
-                    ldmatrix4(qa + k * 32 + 32, a2);
-                    mma_bf16_16x8x16(d1, a2[0], a2[1], a2[2], a2[3], kb[2], kb[3]);
-                } else {
-                    asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(kb[0]), "=r"(kb[1]) : "r"(ka - (lane >> 4) * 32 + k * 32));
+        const int j0 = lo + it * 64, buf = it % L.stages;
+        const uint32_t kv = base + L.data + buf * L.tile;
+        ok = wait_or_abort(base + L.bar + 8 * buf, (it / L.stages) & 1, abort_flag);
+        ok = __syncthreads_and(ok);
+        if (!ok) break;
+        {   // scores of 16 keys over half of the columns
+            float d[MT][2][4];
+#pragma unroll
+            for (int m = 0; m < MT; ++m)
+#pragma unroll
+                for (int j = 0; j < 2; ++j)
+#pragma unroll
+                    for (int c = 0; c < 4; ++c) d[m][j][c] = 0.f;
+            const int kr = key0 + (lane >> 4) * 8 + (lane & 7);
+            const uint32_t qa = base + L.q + (lane & 15) * 128, ka = kv + kr * 128;
+#pragma unroll 4
+            for (int k = k0; k < k1; ++k) {
+                uint32_t kb[4], a[4];
+                const int piece = 2 * k + ((lane >> 3) & 1), qp = 2 * k + (lane >> 4);   // eight columns
+                ldmatrix4(ka + (piece >> 3) * 8192 + (((piece & 7) ^ (kr & 7)) << 4), kb);
+#pragma unroll
+                for (int m = 0; m < MT; ++m) {
+                    ldmatrix4(qa + (qp >> 3) * MT * 2048 + m * 2048 + (((qp & 7) ^ (lane & 7)) << 4), a);
+                    mma_bf16_16x8x16(d[m][0], a[0], a[1], a[2], a[3], kb[0], kb[1]);
+                    mma_bf16_16x8x16(d[m][1], a[0], a[1], a[2], a[3], kb[2], kb[3]);
                 }
-                mma_bf16_16x8x16(d0, a[0], a[1], a[2], a[3], kb[0], kb[1]);
             }
             const float f = p.scale * kLog2e;
 #pragma unroll
-            for (int c = 0; c < 4; ++c) {
-                const int key = warp * 8 + 2 * qd + (c & 1), head = g + (c >> 1) * 8;
-                s_s[head * 68 + key] = j0 + key < hi ? (d0[c] + d1[c]) * f : -INFINITY;
-            }
+            for (int m = 0; m < MT; ++m)
+#pragma unroll
+                for (int j = 0; j < 2; ++j)
+#pragma unroll
+                    for (int c = 0; c < 4; c += 2) {
+                        const int key = key0 + j * 8 + 2 * qd, head = m * 16 + g + (c >> 1) * 8;
+                        *reinterpret_cast<float2*>(s_s + (half * 16 * MT + head) * 68 + key) = make_float2(d[m][j][c] * f, d[m][j][c + 1] * f);
+                    }
         }
         __syncthreads();
+        {                                                    // softmax: 16 / MT threads per head, pairs of keys
+            constexpr int TPH = 16 / MT, N = 32 / TPH;
+            const int head = tid / TPH, sub = tid % TPH;
+            const float *sa = s_s + head * 68 + 2 * sub, *sb = sa + 16 * MT * 68;
+            float2 w[N];
+            const float mo = m_s[head];
+            float mn = mo, sum = 0.f;
 #pragma unroll
-        for (int i = 0; i < 2; ++i) {                        // two heads per warp
-            const int head = warp * 2 + i;
-            const float s0 = s_s[head * 68 + lane], s1 = s_s[head * 68 + 32 + lane], mo = m_s[head];
-            float mx = fmaxf(s0, s1);
+            for (int i = 0; i < N; ++i) {
+                const float2 x = *reinterpret_cast<const float2*>(sa + 2 * TPH * i), y = *reinterpret_cast<const float2*>(sb + 2 * TPH * i);
+                const int key = j0 + 2 * (sub + TPH * i);
+                w[i] = make_float2(key < hi ? x.x + y.x : -INFINITY, key + 1 < hi ? x.y + y.y : -INFINITY);
+                mn = fmaxf(mn, fmaxf(w[i].x, w[i].y));       // finite in the end: the first key of a tile always counts
+            }
 #pragma unroll
-            for (int d = 16; d; d >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, d));
-            const float mn = fmaxf(mo, mx);                  // finite: the first key of a tile always counts
-            const float w0 = exp2f(s0 - mn), w1 = exp2f(s1 - mn), sum = warp_sum(w0 + w1);
-            p_s[head * 72 + lane] = from_f<bf16>(w0), p_s[head * 72 + 32 + lane] = from_f<bf16>(w1);
-            __syncwarp();
-            if (lane == 0) {
+            for (int d = TPH / 2; d; d >>= 1) mn = fmaxf(mn, __shfl_xor_sync(0xffffffffu, mn, d));
+#pragma unroll
+            for (int i = 0; i < N; ++i) {
+                w[i] = make_float2(exp2f(w[i].x - mn), exp2f(w[i].y - mn));
+                sum += w[i].x + w[i].y;
+                *reinterpret_cast<uint32_t*>(p_s + head * 72 + 2 * (sub + TPH * i)) = pack_bf16(w[i].x, w[i].y);
+            }
+#pragma unroll
+            for (int d = TPH / 2; d; d >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, d);
+            if (sub == 0) {
                 const float f = exp2f(mo - mn);
                 f_s[head] = f, m_s[head] = mn, l_s[head] = fmaf(l_s[head], f, sum);
             }
         }
         __syncthreads();
-        const float fa = f_s[g], fb = f_s[g + 8];
+        if (it > 0)
 #pragma unroll
-        for (int i = 0; i < NT; ++i)
+            for (int m = 0; m < MT; ++m) {
+                const float fa = f_s[m * 16 + g], fb = f_s[m * 16 + g + 8];
 #pragma unroll
-            for (int j = 0; j < 2; ++j) acc[i][j][0] *= fa, acc[i][j][1] *= fa, acc[i][j][2] *= fb, acc[i][j][3] *= fb;
+                for (int i = 0; i < NT; ++i)
 #pragma unroll
-        for (int kk = 0; kk < 4; ++kk) {
-            uint32_t a[4];
-            ldmatrix4(base + L.p + (lane & 15) * 144 + kk * 32 + (lane >> 4) * 16, a);
+                    for (int j = 0; j < 2; ++j)
+                        acc[i][m][j][0] *= fa, acc[i][m][j][1] *= fa, acc[i][m][j][2] *= fb, acc[i][m][j][3] *= fb;
+            }
+        const int live = min(4, (hi - j0 + 15) / 16);        // 16-key groups with weights other than zero
+#pragma unroll 1
+        for (int kk = 0; kk < live; ++kk) {
+            uint32_t a[MT][4];
+#pragma unroll
+            for (int m = 0; m < MT; ++m) ldmatrix4(base + L.p + (m * 16 + (lane & 15)) * 144 + kk * 32 + (lane >> 4) * 16, a[m]);
+            const int kr = kk * 16 + (lane & 15);
 #pragma unroll
             for (int i = 0; i < NT; ++i) {
                 const int c = (warp * NT + i) * 16;
-                if (c < p.R) {                               // uniform over the warp; a tile is inside the padded row
+                if (c < p.R) {                               // uniform over the warp
                     uint32_t v[4];
-                    ldmatrix4_trans(base + L.kv + (buf * 64 + kk * 16 + (lane & 15)) * L.stride + (c + (lane >> 4) * 8) * 2, v);
-                    mma_bf16_16x8x16(acc[i][0], a[0], a[1], a[2], a[3], v[0], v[1]);
-                    mma_bf16_16x8x16(acc[i][1], a[0], a[1], a[2], a[3], v[2], v[3]);
+                    const int piece = c / 8 + (lane >> 4);
+                    ldmatrix4_trans(kv + (piece >> 3) * 8192 + kr * 128 + (((piece & 7) ^ (kr & 7)) << 4), v);
+#pragma unroll
+                    for (int m = 0; m < MT; ++m) {
+                        mma_bf16_16x8x16(acc[i][m][0], a[m][0], a[m][1], a[m][2], a[m][3], v[0], v[1]);
+                        mma_bf16_16x8x16(acc[i][m][1], a[m][0], a[m][1], a[m][2], a[m][3], v[2], v[3]);
+                    }
                 }
             }
         }
         __syncthreads();                                     // the buffer, the scores and the weights are used again
+        if (tid == 0 && it + L.stages < tiles) fetch(it + L.stages);
     }
-    __syncthreads();
-    float* part = p.part + (((size_t)row * p.H + h0) * splits + split) * p.R;
-    if (tiles > 0)
+    const int ro = p.R + 8;                                  // row of o_s: eight rows apart in different banks
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
 #pragma unroll
         for (int i = 0; i < NT; ++i)
 #pragma unroll
-            for (int j = 0; j < 2; ++j)
-#pragma unroll
-                for (int c = 0; c < 4; ++c) {
-                    const int r = (warp * NT + i) * 16 + j * 8 + 2 * qd + (c & 1), head = g + (c >> 1) * 8;
-                    if (r < p.R && head < hn) part[(size_t)head * splits * p.R + r] = acc[i][j][c];
+            for (int j = 0; j < 2; ++j) {
+                const int r = (warp * NT + i) * 16 + j * 8 + 2 * qd;   // R is a multiple of 8
+                if (r < p.R) {
+                    float* o = o_s + (m * 16 + g) * ro + r;
+                    *reinterpret_cast<float2*>(o) = make_float2(acc[i][m][j][0], acc[i][m][j][1]);
+                    *reinterpret_cast<float2*>(o + 8 * ro) = make_float2(acc[i][m][j][2], acc[i][m][j][3]);
                 }
-    if (tid < hn) {
-        float* ml = p.ml + (((size_t)row * p.H + h0 + tid) * splits + split) * 2;
-        ml[0] = m_s[tid], ml[1] = l_s[tid];
+            }
+    cluster_arrive();
+    cluster_wait();
+    const int part_at = split / C, parts = splits / C;
+    for (int i = rank * 256 + tid; i < hn * (p.R / 4); i += C * 256) {
+        const int head = i / (p.R / 4), c = (i - head * (p.R / 4)) * 4;
+        const uint32_t at = base + L.data + 4 * (head * ro + c), m_at = base + L.st + 4 * head;
+        float4 o = make_float4(0.f, 0.f, 0.f, 0.f), v[8];
+        float m[8], l[8], top = -INFINITY, sum = 0.f;
+#pragma unroll
+        for (int r = 0; r < 8; ++r)
+            if (r < C) m[r] = ld_cluster(m_at, r), l[r] = ld_cluster(m_at + 128, r), v[r] = ld_cluster4(at, r);
+#pragma unroll
+        for (int r = 0; r < 8; ++r)
+            if (r < C) top = fmaxf(top, m[r]);
+#pragma unroll
+        for (int r = 0; r < 8; ++r)
+            if (r < C) {
+                const float w = m[r] == -INFINITY ? 0.f : exp2f(m[r] - top);
+                o.x = fmaf(w, v[r].x, o.x), o.y = fmaf(w, v[r].y, o.y), o.z = fmaf(w, v[r].z, o.z), o.w = fmaf(w, v[r].w, o.w);
+                sum = fmaf(w, l[r], sum);
+            }
+        const size_t dst = ((size_t)row * p.H + h0 + head) * parts + part_at;
+        st4(p.part + dst * p.R + c, o);
+        if (c == 0) p.ml[2 * dst] = top, p.ml[2 * dst + 1] = sum;
     }
+    cluster_arrive();                                        // nobody leaves while another CTA still reads
+    cluster_wait();
+    if (*abort_flag && tid == 0) atomicExch(&g_decoder_status, DECODER_WAIT_TIMEOUT);
 }
 
 // Joins the ranges' parts, adds the sink to the denominator and multiplies with W_uv: y[row][h][v].  CTAs x = 32 values
-// of one head (y) and row (z); the weights are requested before the wait.
-template <int RW>   // words of 16 bytes per lane and row of W_uv: R <= 256 * RW, a multiple of 8
+// of one head (y) for RB rows (z); the weights are requested before the wait.
+template <int RW, int RB>   // words of 16 bytes per lane and row of W_uv: R <= 256 * RW, a multiple of 8
 __global__ void __launch_bounds__(256) latent_join_kernel(const LatentAttnParams p) {
-    extern __shared__ __align__(16) float latent_join_smem[];   // weights of the ranges [splits], latent [R]
-    __shared__ float inv_s;
+    extern __shared__ __align__(16) float c_s[];             // the latents [RB][R]
     griddep_launch_dependents();
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.y, row = blockIdx.z, R = p.R, splits = p.splits;
-    float *w_s = latent_join_smem, *c_s = w_s + (splits + 3) / 4 * 4;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.y, row0 = blockIdx.z * RB, R = p.R, splits = p.splits, M = p.B * p.T;
     const bf16* w = reinterpret_cast<const bf16*>(p.w_uv) + (size_t)h * p.vdim * R;
     uint4 wv[4][RW];
 #pragma unroll
@@ -396,50 +469,83 @@ __global__ void __launch_bounds__(256) latent_join_kernel(const LatentAttnParams
             wv[i][j] = v < p.vdim && c < R ? ldg_stream_128(w + (size_t)v * R + c) : make_uint4(0, 0, 0, 0);
         }
     griddep_wait();
-    const float* ml = p.ml + ((size_t)row * p.H + h) * splits * 2;
-    if (warp == 0) {
-        const float sink = p.sink[h] * kLog2e;
-        float m = sink;
-        for (int s = lane; s < splits; s += 32) m = fmaxf(m, __ldcg(ml + 2 * s));
+    constexpr int PRE = RB == 1 ? 8 : 4;                     // parts in flight, with their maxima and sums
+    const float sink = p.sink[h] * kLog2e;
+    float o[RB][RW], top[RB], l[RB];
 #pragma unroll
-        for (int d = 16; d; d >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, d));
-        float l = 0.f;
-        for (int s = lane; s < splits; s += 32) {
-            const float e = exp2f(__ldcg(ml + 2 * s) - m);   // 0 for a range without keys (m = -inf)
-            w_s[s] = e;
-            l = fmaf(e, __ldcg(ml + 2 * s + 1), l);
-        }
-        l = warp_sum(l) + exp2f(sink - m);
-        if (lane == 0) inv_s = 1.f / l;
+    for (int b = 0; b < RB; ++b) {
+        top[b] = sink, l[b] = 1.f;
+#pragma unroll
+        for (int j = 0; j < RW; ++j) o[b][j] = 0.f;
     }
-    __syncthreads();
-    const float* part = p.part + ((size_t)row * p.H + h) * splits * R;
-    for (int c = tid; c < R; c += 256) {
-        float o = 0.f;
-#pragma unroll 8
-        for (int s = 0; s < splits; ++s) {
-            const float e = w_s[s];
-            o = fmaf(e, e > 0.f ? __ldcg(part + (size_t)s * R + c) : 0.f, o);
+    for (int s0 = 0; s0 < splits; s0 += PRE) {
+        float2 st[RB][PRE];
+        float v[RB][RW][PRE];
+#pragma unroll
+        for (int b = 0; b < RB; ++b) {
+            const size_t at = ((size_t)min(row0 + b, M - 1) * p.H + h) * splits;
+#pragma unroll
+            for (int s = 0; s < PRE; ++s) {
+                const bool in = s0 + s < splits;
+                st[b][s] = in ? __ldcg(reinterpret_cast<const float2*>(p.ml) + at + s0 + s) : make_float2(-INFINITY, 0.f);
+#pragma unroll
+                for (int j = 0; j < RW; ++j) v[b][j][s] = in && tid + 256 * j < R ? __ldcg(p.part + (at + s0 + s) * R + tid + 256 * j) : 0.f;
+            }
         }
-        c_s[c] = o * inv_s;
+#pragma unroll
+        for (int b = 0; b < RB; ++b) {
+            float m = top[b];
+#pragma unroll
+            for (int s = 0; s < PRE; ++s) m = fmaxf(m, st[b][s].x);
+            const float f = exp2f(top[b] - m);
+            top[b] = m, l[b] *= f;
+#pragma unroll
+            for (int j = 0; j < RW; ++j) o[b][j] *= f;
+#pragma unroll
+            for (int s = 0; s < PRE; ++s) {
+                const float w = exp2f(st[b][s].x - m);       // 0 for a range without keys
+                l[b] = fmaf(w, st[b][s].y, l[b]);
+#pragma unroll
+                for (int j = 0; j < RW; ++j) o[b][j] = fmaf(w, v[b][j][s], o[b][j]);
+            }
+        }
     }
+#pragma unroll
+    for (int b = 0; b < RB; ++b)
+#pragma unroll
+        for (int j = 0; j < RW; ++j)
+            if (tid + 256 * j < R) c_s[b * R + tid + 256 * j] = o[b][j] / l[b];
     __syncthreads();
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
-        float d = 0.f;
+    for (int b = 0; b < RB; ++b) {
+        if (row0 + b >= M) break;
+        float d[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
         for (int j = 0; j < RW; ++j) {
             const int c = (lane + 32 * j) * 8;
             if (c < R) {
-                float f[8];
-                unpack8(wv[i][j], f);
+                const float4 x = *reinterpret_cast<const float4*>(c_s + b * R + c), y = *reinterpret_cast<const float4*>(c_s + b * R + c + 4);
 #pragma unroll
-                for (int e = 0; e < 8; ++e) d = fmaf(f[e], c_s[c + e], d);
+                for (int i = 0; i < 4; ++i) {
+                    float f[8];
+                    unpack8(wv[i][j], f);
+                    d[i] = fmaf(f[0], x.x, fmaf(f[1], x.y, fmaf(f[2], x.z, fmaf(f[3], x.w, d[i]))));
+                    d[i] = fmaf(f[4], y.x, fmaf(f[5], y.y, fmaf(f[6], y.z, fmaf(f[7], y.w, d[i]))));
+                }
             }
         }
-        d = warp_sum(d);
-        const int v = blockIdx.x * 32 + warp * 4 + i;
-        if (lane == 0 && v < p.vdim) reinterpret_cast<bf16*>(p.y)[((size_t)row * p.H + h) * p.vdim + v] = from_f<bf16>(d);
+        // four sums over 32 lanes: sum i ends in the lanes of group i of eight
+#pragma unroll
+        for (int n = 2, s = 16; n; n >>= 1, s >>= 1)
+#pragma unroll
+            for (int i = 0; i < n; ++i) {
+                const float keep = (lane & s) ? d[i + n] : d[i], give = (lane & s) ? d[i] : d[i + n];
+                d[i] = keep + __shfl_xor_sync(0xffffffffu, give, s);
+            }
+#pragma unroll
+        for (int s = 4; s; s >>= 1) d[0] += __shfl_xor_sync(0xffffffffu, d[0], s);
+        const int v = blockIdx.x * 32 + warp * 4 + lane / 8;
+        if (lane % 8 == 0 && v < p.vdim) reinterpret_cast<bf16*>(p.y)[((size_t)(row0 + b) * p.H + h) * p.vdim + v] = from_f<bf16>(d[0]);
     }
 }
 

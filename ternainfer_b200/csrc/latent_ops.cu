@@ -60,11 +60,28 @@ static int wkv_one(const WkvParams& p, int pdl, void* stream) {
     return wkv_one_n<A, 0>(p, dvp, pdl, stream);
 }
 
-static int latent_smem_limit() { return 227 * 1024; }
+constexpr int kLatentSmemLimit = 227 * 1024;
 
+template <int NT, int MT>
+static int latent_step_m(const LatentAttnParams& p, const CUtensorMap& map, int pdl, void* stream) {
+    CUtensorMap map_q;
+    if (!encode_rows(&map_q, p.qa, (long long)p.B * p.T * p.H, p.ld, p.ld, 16 * MT)) return bad(DECODER_LAUNCH, "latent_step: tensor map refused");
+    const dim3 grid(p.splits * p.cluster, (p.H + 16 * MT - 1) / (16 * MT), p.B * p.T);
+    return launch(latent_step_kernel<NT, MT>, grid, 256, (size_t)LatentStepSmem(p.ld, MT, kLatentSmemLimit).total, pdl, stream, p.cluster, p, kLatentSmemLimit, map_q, map);
+}
 template <int NT>
-static int latent_step(const LatentAttnParams& p, int pdl, void* stream) {
-    return launch(latent_step_kernel<NT>, dim3(p.splits, (p.H + 15) / 16, p.B * p.T), 256, (size_t)LatentStepSmem(p.ld).total, pdl, stream, 1, p);
+static int latent_step(const LatentAttnParams& p, const CUtensorMap& map, int pdl, void* stream) {
+    if constexpr (NT <= 4)
+        if (p.H > 16 && LatentStepSmem(p.ld, 2, kLatentSmemLimit).total <= kLatentSmemLimit) return latent_step_m<NT, 2>(p, map, pdl, stream);
+    return latent_step_m<NT, 1>(p, map, pdl, stream);
+}
+
+template <int RW>
+static int latent_join(const LatentAttnParams& p, int pdl, void* stream) {
+    const int M = p.B * p.T;
+    const dim3 grid((p.vdim + 31) / 32, p.H, M);
+    if (M == 1) return launch(latent_join_kernel<RW, 1>, grid, 256, (size_t)p.R * 4, pdl, stream, 1, p);
+    return launch(latent_join_kernel<RW, 4>, dim3(grid.x, grid.y, (M + 3) / 4), 256, (size_t)p.R * 16, pdl, stream, 1, p);
 }
 
 }  // namespace tsp
@@ -93,7 +110,9 @@ extern "C" int decoder_latent_prep(const decoder_latent_prep_args* a, int dtype,
         return bad(DECODER_BAD_SHAPE, "latent_prep: cache layout");
     if (!a->z || !a->cq || !a->q_norm || !a->pos || (a->cache && (!a->kv_norm || (a->dims && !a->trig)))) return bad(DECODER_BAD_POINTER, "latent_prep: null pointer");
     const dim3 grid((unsigned)(a->B * a->T));
-    return dtype ? launch(latent_prep_kernel<float>, grid, 256, 0, pdl, stream, 1, *a) : launch(latent_prep_kernel<bf16>, grid, 256, 0, pdl, stream, 1, *a);
+    const size_t smem = (size_t)(a->q_rank + (a->cache ? a->R + a->rot : 0)) * 4;
+    if (smem > 200 * 1024) return bad(DECODER_BAD_SHAPE, "latent_prep: rows of at most 51200");
+    return dtype ? launch(latent_prep_kernel<float>, grid, 256, smem, pdl, stream, 1, *a) : launch(latent_prep_kernel<bf16>, grid, 256, smem, pdl, stream, 1, *a);
 }
 
 extern "C" int decoder_rotate(const decoder_rotate_args* a, int dtype, int pdl, void* stream) {
@@ -105,12 +124,11 @@ extern "C" int decoder_rotate(const decoder_rotate_args* a, int dtype, int pdl, 
 }
 
 extern "C" int decoder_absorb(const decoder_absorb_args* a, int pdl, void* stream) {
-    if (a->B < 1 || a->T < 1 || a->B * a->T > 8 || a->H < 1 || a->dim < 1 || a->dim > 1024 || a->R < 8 || a->R % 8 || a->rot < 0 || a->dims % 2 || a->dims > a->rot ||
+    if (a->B < 1 || a->T < 1 || a->B * a->T > 8 || a->H < 1 || a->dim < 8 || a->dim % 8 || a->R < 1 || a->rot < 0 || a->rot % 8 || a->dims % 2 || a->dims > a->rot ||
         a->r_at < a->R || a->r_at + a->rot > a->ld)
-        return bad(DECODER_BAD_SHAPE, "absorb: up to 8 rows, R a multiple of 8");
-    if (!a->q || !a->w_uk || !a->qa || !a->pos || misaligned(a->w_uk, 16) || (a->dims && !a->trig)) return bad(DECODER_BAD_POINTER, "absorb: null or misaligned pointer");
-    const size_t smem = ((size_t)(8 * a->dim + 3) / 4 * 4 + (size_t)8 * a->B * a->T * 128) * 4;
-    return launch(absorb_kernel, dim3((a->R + 127) / 128 + 1, a->H), 256, smem, pdl, stream, 1, *a);
+        return bad(DECODER_BAD_SHAPE, "absorb: up to 8 rows, dim and rot multiples of 8");
+    if (!a->q || !a->w_uk_t || !a->qa || !a->pos || misaligned(a->q, 16) || misaligned(a->w_uk_t, 16) || (a->dims && !a->trig)) return bad(DECODER_BAD_POINTER, "absorb: null or misaligned pointer");
+    return launch(absorb_kernel, dim3((a->R + 127) / 128 + 1, a->H), 256, 0, pdl, stream, 1, *a);
 }
 
 static int latent_attn_check(const decoder_latent_attn_args* a) {
@@ -130,25 +148,26 @@ extern "C" int decoder_latent_attn(const decoder_latent_attn_args* a, int dtype,
 
 extern "C" int decoder_latent_step_width(void) {
     int ld = 8;
-    while (LatentStepSmem(ld + 8).total <= latent_smem_limit()) ld += 8;
+    while (LatentStepSmem(ld + 8, 1, kLatentSmemLimit).total <= kLatentSmemLimit) ld += 8;
     return ld;
 }
 
 extern "C" int decoder_latent_step(const decoder_latent_attn_args* a, int pdl, void* stream) {
     if (int rc = latent_attn_check(a)) return rc;
-    if (a->R % 8 || a->R > 1024 || a->splits < 1 || a->splits > 1024 || a->vdim < 1 || LatentStepSmem(a->ld).total > latent_smem_limit())
+    if (a->R % 8 || a->R > 1024 || a->splits < 1 || a->splits > 1024 || a->cluster < 1 || a->cluster > 8 || a->vdim < 1 ||
+        LatentStepSmem(a->ld, 1, kLatentSmemLimit).total > kLatentSmemLimit)
         return bad(DECODER_BAD_SHAPE, "latent_step: R a multiple of 8 up to 1024, rows that fit shared memory");
     if (!a->part || !a->ml || !a->w_uv || !a->y || misaligned(a->w_uv, 16)) return bad(DECODER_BAD_POINTER, "latent_step: null or misaligned pointer");
-    const int rc = a->R <= 128   ? latent_step<1>(*a, pdl, stream)
-                   : a->R <= 256 ? latent_step<2>(*a, pdl, stream)
-                   : a->R <= 512 ? latent_step<4>(*a, pdl, stream)
-                                 : latent_step<8>(*a, pdl, stream);
+    CUtensorMap map;
+    if (!encode_rows(&map, a->cache, (long long)a->B * a->slots, a->ld, a->ld, 32)) return bad(DECODER_LAUNCH, "latent_step: tensor map refused");
+    const int rc = a->R <= 128   ? latent_step<1>(*a, map, pdl, stream)
+                   : a->R <= 256 ? latent_step<2>(*a, map, pdl, stream)
+                   : a->R <= 512 ? latent_step<4>(*a, map, pdl, stream)
+                                 : latent_step<8>(*a, map, pdl, stream);
     if (rc) return rc;
-    const dim3 grid((a->vdim + 31) / 32, a->H, a->B * a->T);
-    const size_t smem = (size_t)((a->splits + 3) / 4 * 4 + a->R) * 4;
-    if (a->R <= 256) return launch(latent_join_kernel<1>, grid, 256, smem, pdl, stream, 1, *a);
-    if (a->R <= 512) return launch(latent_join_kernel<2>, grid, 256, smem, pdl, stream, 1, *a);
-    return launch(latent_join_kernel<4>, grid, 256, smem, pdl, stream, 1, *a);
+    if (a->R <= 256) return latent_join<1>(*a, pdl, stream);
+    if (a->R <= 512) return latent_join<2>(*a, pdl, stream);
+    return latent_join<4>(*a, pdl, stream);
 }
 
 extern "C" int decoder_latent_prompt(const decoder_latent_prompt_args* a, void* stream) {
@@ -194,12 +213,25 @@ extern "C" int decoder_moe_plain(const decoder_moe_args* a, int dtype, int pdl, 
     return dtype ? launch(moe_down_plain_kernel<float>, down, 256, 0, pdl, stream, 1, *a) : launch(moe_down_plain_kernel<bf16>, down, 256, 0, pdl, stream, 1, *a);
 }
 
+template <int P>
+static int moe_up_step(const MoeParams& p, int pdl, void* stream) {
+    const int items = p.ff / 8 * std::min(p.E, p.M * p.top);
+    return launch(moe_up_step_kernel<P>, dim3(std::min(items, 2 * sm_count())), kRowsWarps * 32, (size_t)p.M * (p.K * 2 + 64), pdl, stream, 1, p);
+}
+
 extern "C" int decoder_moe_up_step(const decoder_moe_args* a, int pdl, void* stream) {
     if (int rc = moe_check(a)) return rc;
-    if (a->M > 8 || a->K % 8 || a->gate.kind < 1 || a->gate.kind > 2) return bad(DECODER_BAD_SHAPE, "moe_up_step: M <= 8, K a multiple of 8");
-    if (!a->logits || !a->router_bias || !a->chosen || !a->weight || !a->x || !a->w_up || !a->act || misaligned(a->x, 16) || misaligned(a->w_up, 16))
+    if (a->M > 8 || a->K % 8 || a->K > 12288 || a->gate.kind < 1 || a->gate.kind > 2) return bad(DECODER_BAD_SHAPE, "moe_up_step: M <= 8, K a multiple of 8 up to 12288");
+    if (!a->router || !a->router_bias || !a->chosen || !a->weight || !a->x || !a->w_up || !a->act || misaligned(a->router, 16) || misaligned(a->x, 16) ||
+        misaligned(a->w_up, 16))
         return bad(DECODER_BAD_POINTER, "moe_up_step: null or misaligned pointer");
-    return launch(moe_up_step_kernel, dim3(a->ff / 8, std::min(a->E, a->M * a->top)), kRowsWarps * 32, (size_t)8 * a->E * 4, pdl, stream, 1, *a);
+    const int rc = launch(router_step_kernel, dim3(a->M), 1024, (size_t)a->K * 2 + (size_t)a->E * 4, pdl, stream, 1, *a);
+    if (rc) return rc;
+    // k-steps in flight: what leaves the last batch of a warp's share the fullest
+    const int steps = ((a->K + 31) / 32 + kRowsWarps - 1) / kRowsWarps;
+    const auto waste = [&](int n) { return (steps + n - 1) / n * n - steps; };
+    if (waste(6) <= waste(5) && waste(6) <= waste(4)) return moe_up_step<6>(*a, pdl, stream);
+    return waste(5) <= waste(4) ? moe_up_step<5>(*a, pdl, stream) : moe_up_step<4>(*a, pdl, stream);
 }
 
 extern "C" int decoder_moe_down_step(const decoder_moe_args* a, int pdl, void* stream) {

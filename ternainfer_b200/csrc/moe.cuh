@@ -5,8 +5,8 @@
 //
 // Weights: gate and up rows in blocks of eight in one matrix [E][2 * ff][K] (gate.cuh), down [E][D][ff]; ff padded to a
 // multiple of 8.  Prompts (bf16): rows are sorted by expert and go through the grouped GEMM (group_gemm_tc.cuh); the
-// residual kernel adds the weighted results (hyper.cuh).  Up to eight tokens: one launch routes and makes the
-// activations, expert by expert, so that an expert's weights are read once for all its tokens; a second one sums the
+// residual kernel adds the weighted results (hyper.cuh).  Up to eight tokens: one launch routes, one makes the
+// activations, expert by expert, so that an expert's weights are read once for all its tokens; a third one sums the
 // down projections of all experts, and the mixer's output projection with them, without leaving the registers.
 // Other types and sizes: one warp per output.
 #pragma once
@@ -37,15 +37,12 @@ __device__ __forceinline__ void next_choice(const float* z, int E, int lane, flo
 }
 
 // One warp: the chosen experts of one token and their weights, top <= 32: lane j holds choice j.  z: [E] in shared memory.
-__device__ __forceinline__ void route_token(const MoeParams& p, int token, float* z, int lane, int& expert, float& weight) {
-    const float* logits = p.logits + (size_t)token * p.E;
-    for (int i = lane; i < p.E; i += 32) z[i] = __ldcg(logits + i) + p.router_bias[i];
-    __syncwarp();
+__device__ __forceinline__ void choose(const float* z, int E, int top, int lane, int& expert, float& weight) {
     float v = INFINITY, best = 0.f, mine = 0.f;
     int e = -1;
     expert = 0;
-    for (int j = 0; j < p.top; ++j) {
-        next_choice(z, p.E, lane, v, e);
+    for (int j = 0; j < top; ++j) {
+        next_choice(z, E, lane, v, e);
         if (j == 0) best = v;
         if (lane == j) expert = e, mine = expf(v - best);
     }
@@ -61,7 +58,10 @@ static __global__ void __launch_bounds__(256) route_kernel(const MoeParams p) {
     if (token >= p.M) return;
     int e;
     float w;
-    route_token(p, token, route_smem + (threadIdx.x >> 5) * p.E, lane, e, w);
+    float* z = route_smem + (threadIdx.x >> 5) * p.E;
+    for (int i = lane; i < p.E; i += 32) z[i] = __ldcg(p.logits + (size_t)token * p.E + i) + p.router_bias[i];
+    __syncwarp();
+    choose(z, p.E, p.top, lane, e, w);
     if (lane < p.top) {
         const int i = token * p.top + lane;
         p.chosen[i] = e, p.weight[i] = w;
@@ -149,64 +149,121 @@ __device__ __forceinline__ int distinct_experts(const int* chosen, int n, int E,
     return count;
 }
 
-// act[token * top + j][f]: CTAs x = 16 rows of gate and up (8 activations), y = one of the chosen experts
-static __global__ void __launch_bounds__(kRowsWarps * 32, 2) moe_up_step_kernel(const MoeParams p) {
-    extern __shared__ __align__(16) float moe_step_smem[];   // logits [8][E]
-    __shared__ float part[kRowsWarps][16][9];
-    __shared__ int chosen[8 * kMoeMaxTop], list[8 * kMoeMaxTop], pair_of[8];
+// Router of up to eight tokens: one CTA per token makes the logits, one warp per expert in turn, and chooses.
+static __global__ void __launch_bounds__(1024) router_step_kernel(const MoeParams p) {
+    extern __shared__ __align__(16) uint8_t router_smem[];   // the token's input [K] bf16, logits [E]
+    griddep_launch_dependents();
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, token = blockIdx.x, K = p.K, words = K / 8;
+    const bf16* w = reinterpret_cast<const bf16*>(p.router);
+    uint4* x_s = reinterpret_cast<uint4*>(router_smem);
+    float* z_s = reinterpret_cast<float*>(router_smem + (size_t)words * 16);
+    constexpr int PRE = 8;                                   // words of the warp's first expert that are under way before the wait
+    uint4 wv[PRE];
+#pragma unroll
+    for (int i = 0; i < PRE; ++i) wv[i] = warp < p.E && lane + 32 * i < words ? ldg_stream_128(w + (size_t)warp * K + (lane + 32 * i) * 8) : make_uint4(0, 0, 0, 0);
+    griddep_wait();
+    for (int c = tid; c < words; c += blockDim.x) x_s[c] = __ldcg(reinterpret_cast<const uint4*>(p.x) + (size_t)token * words + c);
+    __syncthreads();
+    for (int e = warp; e < p.E; e += 32) {
+        float z = 0.f;
+        for (int c0 = 0; c0 < words; c0 += 32 * PRE) {
+            if (e != warp || c0)
+#pragma unroll
+                for (int i = 0; i < PRE; ++i) {
+                    const int c = c0 + lane + 32 * i;
+                    wv[i] = c < words ? ldg_stream_128(w + (size_t)e * K + c * 8) : make_uint4(0, 0, 0, 0);
+                }
+#pragma unroll
+            for (int i = 0; i < PRE; ++i) {
+                const int c = c0 + lane + 32 * i;
+                if (c < words) {
+                    float a[8], b[8];
+                    unpack8(wv[i], a), unpack8(x_s[c], b);
+#pragma unroll
+                    for (int j = 0; j < 8; ++j) z = fmaf(a[j], b[j], z);
+                }
+            }
+        }
+        z = warp_sum(z);
+        if (lane == 0) z_s[e] = z + p.router_bias[e];
+    }
+    __syncthreads();
+    if (warp == 0) {
+        int e;
+        float wt;
+        choose(z_s, p.E, p.top, lane, e, wt);
+        if (lane < p.top) p.chosen[token * p.top + lane] = e, p.weight[token * p.top + lane] = wt;
+    }
+}
+
+// act[token * top + j][f].  Work items of 16 rows of gate and up of one chosen expert (8 activations), a contiguous share
+// per CTA; the weights' stream runs on across items, P k-steps per warp ahead.  The inputs lie in shared memory.
+template <int P>
+__global__ void __launch_bounds__(kRowsWarps * 32, 2) moe_up_step_kernel(const MoeParams p) {
+    extern __shared__ __align__(16) uint8_t moe_up_smem[];   // inputs [M][K] bf16, rows 64 bytes longer
+    __shared__ float part[2][kRowsWarps][16][9];
+    __shared__ int chosen[8 * kMoeMaxTop], list[8 * kMoeMaxTop];
     griddep_launch_dependents();
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, q = lane & 3;
-    const int K = p.K, steps = (K + 31) >> 5, top = p.top, n0 = blockIdx.x * 16;
+    const int K = p.K, steps = (K + 31) >> 5, top = p.top, blocks = p.ff / 8, xs = K * 2 + 64;
     const int s0 = steps * warp / kRowsWarps, s1 = steps * (warp + 1) / kRowsWarps;
-    if (tid < 8) pair_of[tid] = -1;
     griddep_wait();
-    if (warp < p.M) {
-        int e;
-        float w;
-        route_token(p, warp, moe_step_smem + warp * p.E, lane, e, w);
-        if (lane < top) {
-            chosen[warp * top + lane] = e;
-            if (blockIdx.x == 0 && blockIdx.y == 0) p.chosen[warp * top + lane] = e, p.weight[warp * top + lane] = w;
-        }
+    for (int i = tid; i < p.M * top; i += blockDim.x) chosen[i] = __ldcg(p.chosen + i);
+    for (int i = tid; i < p.M * (K / 8); i += blockDim.x) {
+        const int t = i / (K / 8), c = i - t * (K / 8);
+        *reinterpret_cast<uint4*>(moe_up_smem + t * xs + c * 16) = __ldcg(reinterpret_cast<const uint4*>(p.x) + i);
     }
     __syncthreads();
     const int n = distinct_experts(chosen, p.M * top, p.E, list);
-    if ((int)blockIdx.y >= n) return;
-    const int e = list[blockIdx.y];
-    for (int i = tid; i < p.M * top; i += blockDim.x)
-        if (chosen[i] == e) pair_of[i / top] = i;
-    __syncthreads();
-    const bf16* w = reinterpret_cast<const bf16*>(p.w_up) + ((size_t)e * 2 * p.ff + n0) * K + q * 8;
-    const bf16 *w0 = w + (size_t)g * K, *w1 = w + (size_t)(g + 8) * K;
-    const bf16* x = reinterpret_cast<const bf16*>(p.x) + (size_t)(g < p.M ? g : 0) * K + q * 8;
-    const bool xok = g < p.M && pair_of[g] >= 0;
+    const int items = n * blocks, i0 = (int)((long long)items * blockIdx.x / gridDim.x), i1 = (int)((long long)items * (blockIdx.x + 1) / gridDim.x);
+    const bf16* w_up = reinterpret_cast<const bf16*>(p.w_up);
     const uint4 zero = make_uint4(0, 0, 0, 0);
-    float acc[4] = {0.f, 0.f, 0.f, 0.f};
-    for (int s = s0; s < s1; s += kRowsPre) {
-        uint4 a[kRowsPre], b[kRowsPre], xv[kRowsPre];
+    const int batches = (s1 - s0 + P - 1) / P;               // per item
+    uint4 a[P], b[P];
+    auto fetch = [&](int u, int item, int batch) {
+        const int s = s0 + batch * P + u;
+        const bool in = item < i1 && s < s1 && 32 * s + q * 8 < K;
+        const bf16* w = w_up;
+        if (in) w += ((size_t)list[item / blocks] * 2 * p.ff + item % blocks * 16 + g) * K + 32 * s + q * 8;
+        a[u] = in ? ldg_stream_128(w) : zero;
+        b[u] = in ? ldg_stream_128(w + (size_t)8 * K) : zero;
+    };
+    int next_item = i0, next_batch = 0;
+    auto advance = [&]() {
+        if (++next_batch >= batches) next_batch = 0, ++next_item;
+    };
 #pragma unroll
-        for (int u = 0; u < kRowsPre; ++u) {
-            const bool in = s + u < s1 && 32 * (s + u) + q * 8 < K;
-            a[u] = in ? ldg_stream_128(w0 + 32 * (s + u)) : zero;
-            b[u] = in ? ldg_stream_128(w1 + 32 * (s + u)) : zero;
-            xv[u] = in && xok ? ld_cg_128(x + 32 * (s + u)) : zero;
+    for (int u = 0; u < P; ++u) fetch(u, next_item, next_batch);
+    advance();
+    const uint8_t* xrow = moe_up_smem + g * xs + q * 16;
+    for (int item = i0; item < i1; ++item) {
+        float acc[4] = {0.f, 0.f, 0.f, 0.f};
+        for (int batch = 0; batch < batches; ++batch) {
+#pragma unroll
+            for (int u = 0; u < P; ++u) {
+                const int s = s0 + batch * P + u;
+                const uint4 xv = g < p.M && s < s1 && 32 * s + q * 8 < K ? *reinterpret_cast<const uint4*>(xrow + 64 * s) : zero;
+                mma_bf16_16x8x16(acc, a[u].x, b[u].x, a[u].y, b[u].y, xv.x, xv.y);
+                mma_bf16_16x8x16(acc, a[u].z, b[u].z, a[u].w, b[u].w, xv.z, xv.w);
+                fetch(u, next_item, next_batch);
+            }
+            advance();
         }
+        float (*pt)[16][9] = part[(item - i0) & 1];          // written again two items later, behind a barrier
+        pt[warp][g][2 * q] = acc[0], pt[warp][g][2 * q + 1] = acc[1];
+        pt[warp][g + 8][2 * q] = acc[2], pt[warp][g + 8][2 * q + 1] = acc[3];
+        __syncthreads();
+        if (tid < 128) {
+            const int r = tid & 15, t = tid >> 4, e = list[item / blocks];
+            float v = 0.f;
 #pragma unroll
-        for (int u = 0; u < kRowsPre; ++u) {
-            mma_bf16_16x8x16(acc, a[u].x, b[u].x, a[u].y, b[u].y, xv[u].x, xv[u].y);
-            mma_bf16_16x8x16(acc, a[u].z, b[u].z, a[u].w, b[u].w, xv[u].z, xv[u].w);
+            for (int i = 0; i < kRowsWarps; ++i) v += pt[i][r][t];
+            const float up = __shfl_down_sync(0xffffffffu, v, 8);
+            int pair = -1;
+            for (int j = 0; t < p.M && j < top; ++j)
+                if (chosen[t * top + j] == e) pair = t * top + j;
+            if (r < 8 && pair >= 0) reinterpret_cast<bf16*>(p.act)[(size_t)pair * p.ff + item % blocks * 8 + r] = from_f<bf16>(gated(v, up, p.gate));
         }
-    }
-    part[warp][g][2 * q] = acc[0], part[warp][g][2 * q + 1] = acc[1];
-    part[warp][g + 8][2 * q] = acc[2], part[warp][g + 8][2 * q + 1] = acc[3];
-    __syncthreads();
-    if (tid < 128) {
-        const int r = tid & 15, t = tid >> 4;
-        float v = 0.f;
-#pragma unroll
-        for (int i = 0; i < kRowsWarps; ++i) v += part[i][r][t];
-        const float up = __shfl_down_sync(0xffffffffu, v, 8);
-        if (r < 8 && pair_of[t] >= 0) reinterpret_cast<bf16*>(p.act)[(size_t)pair_of[t] * p.ff + n0 / 2 + r] = from_f<bf16>(gated(v, up, p.gate));
     }
 }
 

@@ -267,12 +267,21 @@ static __global__ void __launch_bounds__(256) wkv_carry_kernel(const WkvParams p
     const size_t unit = blockIdx.y, words = (size_t)n + p.dk;
     float* part = p.part + unit * p.n_seg * words;
     float s = p.pos[0] == 0 ? 0.f : ld_cg(p.state + unit * n + e);
-    for (int i = 0; i < p.n_seg; ++i) {
-        float* at = part + i * words;
-        const bool last = i == p.n_seg - 1;
-        const float own = last ? 0.f : ld_cg(at + e), w = last ? 0.f : ld_cg(at + n + e / p.dv);
-        at[e] = s;
-        s = fmaf(w, s, own);
+    constexpr int U = 8;                                     // segments in flight
+    for (int i = 0; i < p.n_seg; i += U) {
+        float own[U], w[U];
+#pragma unroll
+        for (int j = 0; j < U; ++j) {
+            const bool in = i + j < p.n_seg - 1;             // nothing follows the last segment
+            const float* at = part + (size_t)(in ? i + j : 0) * words;
+            own[j] = in ? ld_cg(at + e) : 0.f, w[j] = in ? ld_cg(at + n + e / p.dv) : 0.f;
+        }
+#pragma unroll
+        for (int j = 0; j < U; ++j)
+            if (i + j < p.n_seg) {
+                part[(size_t)(i + j) * words + e] = s;
+                s = fmaf(w[j], s, own[j]);
+            }
     }
 }
 

@@ -142,6 +142,14 @@ def gated(z, bias, gate: Gate) -> torch.Tensor:
     return out
 
 
+def gated_linear(x, weight, bias, gate: Gate) -> torch.Tensor:
+    """Activation of a gated feed-forward from its input: x [M, K], weight [2n, K] and bias in blocks of 8 gate and 8 up
+    rows -> [M, n]; bf16 in one launch (tcgen05, the gate in the epilogue), otherwise the vendor GEMM and the gate."""
+    if x.dtype == torch.bfloat16 and x.shape[1] % 8 == 0:
+        return group_gemm(x, weight[None], bias=bias, gate=gate)
+    return gated(linear(x, weight), bias, gate)
+
+
 def group_gemm(x, weight, counts=None, bias=None, gate: Gate = NO_GATE) -> torch.Tensor:
     """bf16 rows sorted by group times their group's weights [groups, N, K] (tcgen05); ``counts`` int32 [groups]: rows of
     every group, None for a single group.  ``gate`` as in ``rows_linear``."""
@@ -285,12 +293,13 @@ def rotate(src, dst, heads: int, off_src: int, off_dst: int, rot: int, trig, pos
     check(load_decoder_library().decoder_rotate(ctypes.byref(a), _dtype(src), int(step), _stream()))
 
 
-def absorb(q, w_uk, heads: int, dim: int, rot: int, r_at: int, ld: int, trig, pos, T: int, step: bool = False) -> torch.Tensor:
-    """Queries [M, heads * (dim + rot)] to the cache's layout [M, heads, ld]: W_uk^T q_u in front, the rotated part from r_at."""
+def absorb(q, w_uk, w_uk_t, heads: int, dim: int, rot: int, r_at: int, ld: int, trig, pos, T: int, step: bool = False) -> torch.Tensor:
+    """Queries [M, heads * (dim + rot)] to the cache's layout [M, heads, ld]: W_uk^T q_u in front, the rotated part from r_at.
+    ``w_uk`` [heads * dim, R], ``w_uk_t`` [heads, R, dim] the same head by head transposed."""
     M, R = q.shape[0], w_uk.shape[1]
-    if few_rows(q) and R % 8 == 0:
+    if few_rows(q) and dim % 8 == 0 and rot % 8 == 0:
         qa = torch.empty((M, heads, ld), dtype=q.dtype, device=q.device)
-        a = AbsorbArgs(q.data_ptr(), w_uk.data_ptr(), qa.data_ptr(), _ptr(trig), pos.data_ptr(), M // T, T, heads, dim, rot,
+        a = AbsorbArgs(q.data_ptr(), w_uk_t.data_ptr(), qa.data_ptr(), _ptr(trig), pos.data_ptr(), M // T, T, heads, dim, rot,
                        0 if trig is None else trig.shape[1], R, r_at, ld)
         check(load_decoder_library().decoder_absorb(ctypes.byref(a), int(step), _stream()))
         return qa
@@ -304,18 +313,21 @@ def latent_step_fits(R: int, ld: int) -> bool:
     return R % 8 == 0 and R <= 1024 and ld <= load_decoder_library().decoder_latent_step_width()
 
 
-def latent_attention_step(qa, cache, w_uv, sink, pos, T: int, vdim: int, scale: float, step: bool = False, splits: Optional[int] = None):
-    """Absorbed attention of bf16 queries [M, H, ld] over the cache and the product with W_uv: [M, H*vdim]."""
+def latent_attention_step(qa, cache, w_uv, sink, pos, T: int, vdim: int, scale: float, step: bool = False, splits=None):
+    """Absorbed attention of bf16 queries [M, H, ld] over the cache and the product with W_uv: [M, H*vdim].  ``splits``:
+    (clusters, CTAs per cluster) over which the keys of a row are cut."""
     M, H, ld = qa.shape
     R, slots = w_uv.shape[1], cache.shape[1]
     if splits is None:      # as many ranges of at least 32 keys as the chip holds at a time
         sms = torch.cuda.get_device_properties(qa.device).multi_processor_count
-        splits = max(1, min(sms // (M * -(-H // 16)), -(-slots // 32)))
-    part = torch.empty((M, H, splits, R), dtype=torch.float32, device=qa.device)
-    ml = torch.empty((M, H, splits, 2), dtype=torch.float32, device=qa.device)
+        ranges = max(1, min(sms // (M * -(-H // 32)), -(-slots // 32)))
+        splits = (ranges // min(4, ranges), min(4, ranges))
+    parts, cluster = splits
+    part = torch.empty((M, H, parts, R), dtype=torch.float32, device=qa.device)
+    ml = torch.empty((M, H, parts, 2), dtype=torch.float32, device=qa.device)
     y = torch.empty((M, H * vdim), dtype=qa.dtype, device=qa.device)
     a = LatentAttnArgs(qa.data_ptr(), cache.data_ptr(), sink.data_ptr(), pos.data_ptr(), None, w_uv.data_ptr(), part.data_ptr(), ml.data_ptr(),
-                       y.data_ptr(), M // T, T, H, R, ld, vdim, slots, splits, scale)
+                       y.data_ptr(), M // T, T, H, R, ld, vdim, slots, parts, cluster, scale)
     _dtype(qa)
     check(load_decoder_library().decoder_latent_step(ctypes.byref(a), int(step), _stream()))
     return y
@@ -327,7 +339,7 @@ def latent_attention_plain(qa, cache, w_uv, sink, pos, T: int, vdim: int, scale:
     R, slots = w_uv.shape[1], cache.shape[1]
     out = torch.empty((M, H, R), dtype=qa.dtype, device=qa.device)
     a = LatentAttnArgs(qa.data_ptr(), cache.data_ptr(), sink.data_ptr(), pos.data_ptr(), out.data_ptr(), None, None, None, None, M // T, T, H, R, ld,
-                       vdim, slots, 0, scale)
+                       vdim, slots, 0, 0, scale)
     check(load_decoder_library().decoder_latent_attn(ctypes.byref(a), _dtype(qa), int(step), _stream()))
     return torch.bmm(out.transpose(0, 1), w_uv.view(H, vdim, R).transpose(1, 2)).transpose(0, 1).reshape(M, H * vdim)
 
@@ -368,10 +380,10 @@ def expert_step(x, router, router_bias, top: int, w_up, gate: Gate, step: bool =
     """Up to 8 bf16 rows: routing and the chosen experts' activations [M, top, ff], with the choices [M, top] and weights."""
     M, K = x.shape
     E, ff = w_up.shape[0], w_up.shape[1] // 2
-    logits = linear_fp32(x, router, step)
     chosen, weight = _choices(M, top, x.device)
     act = torch.empty((M, top, ff), dtype=x.dtype, device=x.device)
-    a = _moe(M, E, top, K, ff, gate=gate, logits=logits, router_bias=router_bias, chosen=chosen, weight=weight, x=x, w_up=w_up, act=act)
+    a = _moe(M, E, top, K, ff, gate=gate, router=router, router_bias=router_bias, chosen=chosen, weight=weight, x=x, w_up=w_up, act=act)
+    _dtype(x)
     check(load_decoder_library().decoder_moe_up_step(ctypes.byref(a), int(step), _stream()))
     return act, chosen, weight
 

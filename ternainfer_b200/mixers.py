@@ -194,6 +194,7 @@ class LatentAttention(nn.Module):
         self.proj = FusedProjection({n: w[n] for n in ("dq", "dkv") if n in w}, dtype)
         self.uq, self.o = _param(w["uq"], dtype), _param(w["o"], dtype)
         self.ukv = _param(torch.cat([w["uk"], w["uv"]]), dtype)
+        self.uk_t = _param(w["uk"].view(heads, dim, kv_rank).transpose(1, 2), dtype)
         self.q_norm, self.sink = _param(w["dq.norm"]), _param(w["sink"])
         self.kv_norm = _param(w["dkv.norm"]) if self.own else None
         self.register_buffer("trig", rot.table(max_seq_len), persistent=False)
@@ -211,7 +212,7 @@ class LatentAttention(nn.Module):
         if bf16 and T > ops.ROWS and start is not None and ops.latent_prompt_fits(d, r, dv):
             ops.rotate(q, q, H, d, d, r, self.trig, pos, T)
             return ops.latent_attention_prompt(q, self.ukv, cache, self.sink, start, T, H, d, r, dv, self.r_at, self.scale)
-        qa = ops.absorb(q, self.ukv[:H * d], H, d, r, self.r_at, self.ld, self.trig, pos, T, step)
+        qa = ops.absorb(q, self.ukv[:H * d], self.uk_t, H, d, r, self.r_at, self.ld, self.trig, pos, T, step)
         few = bf16 and T <= ops.ROWS and ops.latent_step_fits(self.kv_rank, self.ld)
         return (ops.latent_attention_step if few else ops.latent_attention_plain)(qa, cache, w_uv, self.sink, pos, T, dv, self.scale, step)
 
@@ -249,7 +250,7 @@ class GatedFeedForward(nn.Module):
         if ops.few_rows(h) and (a is None or a.shape[1] % 8 == 0):
             act = ops.rows_linear(h, self.up, self.up_bias, self.gate, step=step)
             return {"y": ops.down_step(act, self.down, self.down_bias, rest=a, w_rest=w_rest, step=step)}
-        act = ops.gated(ops.linear(h, self.up, step=step), self.up_bias, self.gate)
+        act = ops.gated_linear(h, self.up, self.up_bias, self.gate)
         y = torch.addmm(self.down_bias.to(act.dtype), act, self.down.t())
         return {"y": y} if a is None else {"y": ops.linear(a, w_rest, step=step), "y2": y}
 
@@ -267,7 +268,7 @@ class ExpertFeedForward(nn.Module):
 
     def forward(self, h, rest=None, step: bool = False) -> dict:
         a, w_rest = rest or (None, None)
-        if ops.few_rows(h) and (a is None or a.shape[1] % 8 == 0):
+        if ops.few_rows(h) and h.shape[1] <= 12288 and (a is None or a.shape[1] % 8 == 0):
             act, chosen, weight = ops.expert_step(h, self.router, self.router_bias, self.top, self.up, self.gate, step)
             return {"y": ops.down_step(act, self.down, None, chosen, weight, a, w_rest, step)}
         out, slots, weight = ops.expert_rows(h, self.router, self.router_bias, self.top, self.up, self.down, self.gate)

@@ -107,7 +107,7 @@ def attn_got(case, parts, slots=None, path=None, stale=3.0, splits=None):
         if kind == "prompt":
             y = ops.latent_attention_prompt(q, torch.cat([uk, uv]), cache, sink, a, n, H, dim, rot, vdim, r_at, case["scale"])
         else:
-            qa = ops.absorb(q, uk, H, dim, rot, r_at, ld, None, pos(a, b), n)
+            qa = ops.absorb(q, uk, uk.view(H, dim, R).transpose(1, 2).contiguous(), H, dim, rot, r_at, ld, None, pos(a, b), n)
             if kind == "step":
                 y = ops.latent_attention_step(qa, cache, uv, sink, pos(a, b), n, vdim, case["scale"], splits=splits)
             else:
@@ -158,7 +158,7 @@ def test_latent_attention_far_keys_and_tile_borders(dec):
         for parts in ([(0, T)], [(0, 600), (600, 720)], cuts(699, [130]) + singles(699, T), cuts(T, [8]), [(0, 703), (703, 705), (705, T)]):
             got = attn_got(case, parts, slots=T + 40)[0]
             assert rel_rms(got[rows], want[rows]) < 2 * TOL[dtype], parts[:3]
-    for splits in (1, 2, 7, 30, 200):                      # more ranges than keys too
+    for splits in ((1, 1), (1, 2), (7, 1), (3, 8), (30, 7), (1, 8)):                      # more ranges than keys too
         got = attn_got(case, cuts(T, [8]), splits=splits)[0]
         assert rel_rms(got[rows], want[rows]) < 2 * TOL[dtype]
 
@@ -244,21 +244,23 @@ def test_norms_rotation_and_append(dec, rot, dtype):
 
 
 @pytest.mark.parametrize("M,T", [(1, 1), (8, 1), (6, 3), (8, 8)])
-@pytest.mark.parametrize("dim,R", [(128, 512), (48, 136), (7, 8), (130, 40)])
+@pytest.mark.parametrize("dim,R", [(128, 512), (48, 136), (7, 8), (136, 40), (256, 20)])
 def test_absorbed_queries(dec, M, T, dim, R):
     from ternainfer_b200 import decoder_ops as ops
     from ternainfer_b200.sidirax import _parse_rotation
     rot = {"dims": 8, "base": 300.0}
     g = torch.Generator().manual_seed(0)
-    H, rd, B = 3, 10, M // T
+    H, rd, B = 3, 16, M // T
     q, uk = torch.randn((M, H * (dim + rd)), generator=g).bfloat16(), (torch.randn((H * dim, R), generator=g) / dim ** 0.5).bfloat16()
-    ld = R + 16
-    qa = ops.absorb(q.cuda(), uk.cuda(), H, dim, rd, R, ld, _parse_rotation(rot, "t").table(60).cuda(), pos(31, 31 + T), T).double().cpu()
+    r_at = -(-R // 8) * 8
+    ld = r_at + 24
+    qa = ops.absorb(q.cuda(), uk.cuda(), uk.cuda().view(H, dim, R).transpose(1, 2).contiguous(), H, dim, rd, r_at, ld, _parse_rotation(rot, "t").table(60).cuda(), pos(31, 31 + T), T).double().cpu()
     qh = q.view(B, T, H, dim + rd).double()
     want = torch.einsum("bthd,hdr->bthr", qh[..., :dim], uk.view(H, dim, R).double())
     assert rel_rms(qa[:, :, :R].reshape(M, -1), want.reshape(M, -1)) < 4e-3
     turned = torch.stack([o.rotate(qh[b, ..., dim:], range(31, 31 + T), rot) for b in range(B)])
-    assert rel_rms(qa[:, :, R:R + rd].reshape(M, -1), turned.reshape(M, -1)) < 4e-3 and (qa[:, :, R + rd:] == 0).all()
+    assert rel_rms(qa[:, :, r_at:r_at + rd].reshape(M, -1), turned.reshape(M, -1)) < 4e-3
+    assert (qa[:, :, R:r_at] == 0).all() and (qa[:, :, r_at + rd:] == 0).all()
 
 
 # ------------------------------------------------------------------------------- wkv recurrence
@@ -462,7 +464,7 @@ FFS = [dense(56, 0.8), dense(30, 3.0), dense(264, 1.5), moe(5, 2, 24), moe(4, 4,
 @pytest.mark.parametrize("cfg", FFS, ids=lambda c: "-".join(str(x) for v in c.values() for x in (v.values() if isinstance(v, dict) else [v])))
 def test_feed_forwards(dec, cfg, dtype):
     """Few rows and many, with another product in the same residual update and without, widths that suit the kernels and not."""
-    for D, M in ((48, 1), (48, 5), (48, 8), (48, 9), (272, 140), (42, 3), (42, 20), (200, 33)):
+    for D, M in ((48, 1), (48, 5), (48, 8), (48, 9), (272, 140), (42, 3), (42, 20), (200, 33), (2568, 8), (1296, 2)):
         w = ff_weights(cfg, D, dtype)
         f = ff_module(cfg, w, dtype)
         g = torch.Generator().manual_seed(M)
@@ -542,7 +544,7 @@ def test_bad_calls_are_refused_on_the_host(dec):
     assert dec.decoder_wkv(ref(WkvArgs(B=1, T=1, H=1, dk=300, dv=300, rank=1)), 0, 0, None) == 1
     assert dec.decoder_wkv(ref(WkvArgs(B=1, T=40, H=1, dk=8, dv=8, rank=1, n_seg=2, seg_len=16)), 0, 0, None) == 1
     assert dec.decoder_wkv(ref(WkvArgs(B=1, T=1, H=1, dk=8, dv=8, rank=1)), 0, 0, None) == 2
-    assert dec.decoder_latent_step(ref(LatentAttnArgs(B=1, T=1, H=1, R=8, ld=16, slots=4, vdim=8, splits=1)), 0, None) == 2
+    assert dec.decoder_latent_step(ref(LatentAttnArgs(B=1, T=1, H=1, R=8, ld=16, slots=4, vdim=8, splits=1, cluster=1)), 0, None) == 2
     assert dec.decoder_group_gemm(ref(GroupGemmArgs(rows=4, groups=1, N=8, K=8)), None) == 1
     assert dec.decoder_moe_route(ref(MoeArgs(M=1, E=4, top=5, K=8, ff=8)), 0, None) == 1
     with pytest.raises(DecoderOpsError):
