@@ -195,7 +195,7 @@ static int moe_check(const decoder_moe_args* a) {
 extern "C" int decoder_moe_route(const decoder_moe_args* a, int pdl, void* stream) {
     if (int rc = moe_check(a)) return rc;
     if (!a->logits || !a->router_bias || !a->chosen || !a->weight) return bad(DECODER_BAD_POINTER, "moe_route: null pointer");
-    int rc = launch(route_kernel, dim3((a->M + 7) / 8), 256, (size_t)8 * a->E * 4, pdl, stream, 1, *a);
+    int rc = launch(route_kernel, dim3((a->M + 31) / 32), 1024, (size_t)33 * a->E * 4, pdl, stream, 1, *a);
     if (rc || !a->counts) return rc;
     if (a->K % 8) return bad(DECODER_BAD_SHAPE, "moe_route: K a multiple of 8");
     if (!a->rank || !a->slots || !a->x || !a->sorted || misaligned(a->x, 16) || misaligned(a->sorted, 16)) return bad(DECODER_BAD_POINTER, "moe_route: null or misaligned pointer");

@@ -49,24 +49,34 @@ __device__ __forceinline__ void choose(const float* z, int E, int top, int lane,
     weight = mine / warp_sum(mine);
 }
 
-// chosen, weights; with counts also every choice's place among its expert's
-static __global__ void __launch_bounds__(256) route_kernel(const MoeParams p) {
-    extern __shared__ __align__(16) float route_smem[];      // [8][E]
+// chosen, weights; with counts also every choice's place among its expert's: places inside the CTA's 32 tokens first, then
+// one addition per CTA and expert
+static __global__ void __launch_bounds__(1024) route_kernel(const MoeParams p) {
+    extern __shared__ __align__(16) float route_smem[];      // logits [32][E], choices per expert [E]
     griddep_launch_dependents();
     griddep_wait();
-    const int lane = threadIdx.x & 31, token = blockIdx.x * 8 + (threadIdx.x >> 5);
-    if (token >= p.M) return;
-    int e;
-    float w;
-    float* z = route_smem + (threadIdx.x >> 5) * p.E;
-    for (int i = lane; i < p.E; i += 32) z[i] = __ldcg(p.logits + (size_t)token * p.E + i) + p.router_bias[i];
-    __syncwarp();
-    choose(z, p.E, p.top, lane, e, w);
-    if (lane < p.top) {
-        const int i = token * p.top + lane;
-        p.chosen[i] = e, p.weight[i] = w;
-        if (p.counts) p.rank[i] = atomicAdd(p.counts + e, 1);
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, token = blockIdx.x * 32 + warp, E = p.E;
+    int* count = reinterpret_cast<int*>(route_smem + 32 * E);
+    for (int i = tid; i < E; i += 1024) count[i] = 0;
+    int e = 0, rank = 0;
+    float w = 0.f;
+    if (token < p.M) {
+        float* z = route_smem + warp * E;
+        for (int i = lane; i < E; i += 32) z[i] = __ldcg(p.logits + (size_t)token * E + i) + p.router_bias[i];
+        __syncwarp();
+        choose(z, E, p.top, lane, e, w);
     }
+    const bool mine = token < p.M && lane < p.top;
+    const int i = token * p.top + lane;
+    if (mine) p.chosen[i] = e, p.weight[i] = w;
+    if (!p.counts) return;
+    __syncthreads();
+    if (mine) rank = atomicAdd(count + e, 1);
+    __syncthreads();
+    for (int j = tid; j < E; j += 1024)
+        if (count[j]) count[j] = atomicAdd(p.counts + j, count[j]);
+    __syncthreads();
+    if (mine) p.rank[i] = count[e] + rank;
 }
 
 // Rows sorted by expert: one warp per choice finds its slot and copies the token's row there.
@@ -84,7 +94,15 @@ static __global__ void __launch_bounds__(256) sort_rows_kernel(const MoeParams p
     if (lane == 0) p.slots[i] = slot;
     const bf16* src = reinterpret_cast<const bf16*>(p.x) + (size_t)(i / p.top) * p.K;
     bf16* dst = reinterpret_cast<bf16*>(p.sorted) + (size_t)slot * p.K;
-    for (int c = lane; c < p.K / 8; c += 32) stg_128(dst + c * 8, ld_cg_128(src + c * 8));
+    for (int c0 = lane; c0 < p.K / 8; c0 += 32 * 8) {        // eight loads in flight
+        uint4 v[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+            if (c0 + 32 * j < p.K / 8) v[j] = __ldcg(reinterpret_cast<const uint4*>(src) + c0 + 32 * j);
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+            if (c0 + 32 * j < p.K / 8) stg_128(dst + (c0 + 32 * j) * 8, v[j]);
+    }
 }
 
 // ------------------------------------------------------------------------------------------ any type, any size

@@ -235,8 +235,8 @@ def sigmoid_attention(proj, offsets, q_norm, k_norm, bias, slope, cache, pos, T:
 # ------------------------------------------------------------------------------- wkv recurrence
 
 def wkv_segments(T: int, units: int, sms: int):
-    """(segments, tokens per segment) of a prompt portion: enough walks side by side to fill the chip a few times over, each
-    long enough that its initial state does not cost more than itself."""
+    """(segments, tokens per segment) of a prompt portion for ``units`` walks side by side: two rounds of two resident
+    walks per SM, each segment long enough that its initial state does not cost more than itself."""
     want = max(1, min(4 * sms // max(1, units), T // 64))
     length = -(-(-(-T // want)) // 16) * 16
     return -(-T // length), length
@@ -258,7 +258,8 @@ def wkv(r, k, v, g, t1, w2, w0, u, norm, state, pos, T: int, eps: float, step: b
             zw = decay_projection(t1, 0, w2, step)
         o = torch.empty((B * T, H * dv), dtype=torch.float32, device=r.device)
         sms = torch.cuda.get_device_properties(r.device).multi_processor_count
-        n_seg, seg_len = segments or wkv_segments(T, B * H * -(-dv // 64), sms)
+        columns = 32 if dk <= 32 or 64 < dk <= 128 else 64 if dk <= 64 else 16      # of the state per walk
+        n_seg, seg_len = segments or wkv_segments(T, B * H * -(-dv // columns), sms)
         if n_seg > 1:
             part = torch.empty((B, H, n_seg, dk * dv + dk), dtype=torch.float32, device=r.device)
     a = WkvArgs(r.data_ptr(), k.data_ptr(), v.data_ptr(), g.data_ptr(), t1.data_ptr(), _ptr(zw), w2.data_ptr(), w0.data_ptr(), u.data_ptr(),
@@ -321,7 +322,8 @@ def latent_attention_step(qa, cache, w_uv, sink, pos, T: int, vdim: int, scale: 
     if splits is None:      # as many ranges of at least 32 keys as the chip holds at a time
         sms = torch.cuda.get_device_properties(qa.device).multi_processor_count
         ranges = max(1, min(sms // (M * -(-H // 32)), -(-slots // 32)))
-        splits = (ranges // min(4, ranges), min(4, ranges))
+        cluster = min(8 if M * -(-H // 32) * ranges <= 64 else 4, ranges)    # few CTAs: larger clusters still find room
+        splits = (ranges // cluster, cluster)
     parts, cluster = splits
     part = torch.empty((M, H, parts, R), dtype=torch.float32, device=qa.device)
     ml = torch.empty((M, H, parts, 2), dtype=torch.float32, device=qa.device)
@@ -429,5 +431,5 @@ def expert_rows(x, router, router_bias, top: int, w_up, w_down, gate: Gate, plai
     rows = torch.empty((M * top, K), dtype=x.dtype, device=x.device)
     a = _moe(M, E, top, K, ff, logits=logits, router_bias=router_bias, chosen=chosen, weight=weight, counts=counts, rank=rank, slots=slots, x=x,
              sorted=rows)
-    check(lib.decoder_moe_route(ctypes.byref(a), 0, _stream()))
+    check(lib.decoder_moe_route(ctypes.byref(a), 1, _stream()))
     return group_gemm(group_gemm(rows, w_up, counts, gate=gate), w_down, counts), slots, weight
