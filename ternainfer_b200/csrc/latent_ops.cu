@@ -250,7 +250,7 @@ extern "C" int decoder_group_gemm(const decoder_group_gemm_args* a, void* stream
         return bad(DECODER_BAD_SHAPE, "group_gemm: N a multiple of 16, K of 8");
     if (!a->a || !a->w || !a->out || misaligned(a->a, 16) || misaligned(a->w, 16) || misaligned(a->out, 16)) return bad(DECODER_BAD_POINTER, "group_gemm: null or misaligned pointer");
     CUtensorMap ma, mw;
-    if (!encode_rows(&ma, a->a, a->rows, a->K, a->K, 128) || !encode_rows(&mw, a->w, (long long)a->groups * a->N, a->K, a->K, 256))
+    if (!encode_rows(&ma, a->a, a->rows, a->K, a->K, 32) || !encode_rows(&mw, a->w, (long long)a->groups * a->N, a->K, a->K, 128))
         return bad(DECODER_LAUNCH, "group_gemm: tensor map refused");
-    return launch(group_gemm_kernel, dim3(sm_count()), GroupGemmSmem::threads, (size_t)GroupGemmSmem::total, 0, stream, 1, *a, ma, mw);
+    return launch(group_gemm_kernel, dim3(sm_count() & ~1), GroupGemmSmem::threads, (size_t)GroupGemmSmem::total, 0, stream, 2, *a, ma, mw);
 }
