@@ -7,10 +7,13 @@
 
 namespace tsp {
 
+// FAST: the logistic function with the approximate reciprocal
+template <bool FAST = false>
 __device__ __forceinline__ float gated(float g, float u, const decoder_gate& s) {
-    if (s.kind == 1) return g * sigmoid_f(g) * u;
+    const auto sigma = [](float z) { return FAST ? sigmoid_fast(z) : sigmoid_f(z); };
+    if (s.kind == 1) return g * sigma(g) * u;
     g = fminf(g, s.limit), u = fminf(fmaxf(u, -s.limit), s.limit);
-    return g * sigmoid_f(s.alpha * g) * (u + 1.f);
+    return g * sigma(s.alpha * g) * (u + 1.f);
 }
 
 // z [rows][2 * n] in blocks of 8 gate and 8 up columns, bias alike -> out [rows][n]

@@ -146,29 +146,36 @@ __global__ void __launch_bounds__(GroupGemmSmem::threads, 1)
             const float bias = p.bias && w0 + lane < p.N ? p.bias[(size_t)grp * p.N + w0 + lane] : 0.f;
             const int c0 = side * (t.nt / 2), cols = w0 < p.N ? max(0, min(t.nt / 2, t.end - t.row - c0)) : 0;
 #pragma unroll 1
-            for (int c = 0; c < cols; c += 16) {
-                int v[16];
-                tmem_ld16(tmem + lanes + 256 * (n & 1) + c0 + c, v);
-                __syncwarp();                                // the staging of the slice before has been read
-                if (act) {
+            for (int c32 = 0; c32 < cols; c32 += 32) {       // (the tile's half is a multiple of 32)
+                uint32_t v[32];
+                tmem_ld32(tmem + lanes + 256 * (n & 1) + c0 + c32, v);
 #pragma unroll
-                    for (int i = 0; i < 16; ++i) {
-                        const float z = __int_as_float(v[i]) + bias, up = __shfl_down_sync(0xffffffffu, z, 8);
-                        if (!(lane & 8)) sts_b16(st + i * 32 + (lane >> 4) * 16 + (lane & 7) * 2, __bfloat16_as_ushort(__float2bfloat16_rn(gated(z, up, p.gate))));
-                    }
-                    __syncwarp();
-                    const int r = lane >> 1, f = w0 / 2 + (lane & 1) * 8;
-                    if (c + r < cols && f < ldo)
-                        stg_128(reinterpret_cast<bf16*>(p.out) + (size_t)(t.row + c0 + c + r) * ldo + f, lds128(st + r * 32 + (lane & 1) * 16));
-                } else {
+                for (int h = 0; h < 32; h += 16) {
+                    const int c = c32 + h;
+                    __syncwarp();                            // the staging of the slice before has been read
+                    if (act) {                               // of two rows of A, the lane with the gate takes one and the lane with up the other
+                        const bool hi = lane & 8;
+                        const uint32_t at = st + (hi ? 32 : 0) + (lane >> 4) * 16 + (lane & 7) * 2;
 #pragma unroll
-                    for (int i = 0; i < 16; ++i) sts_b16(st + i * 64 + lane * 2, __bfloat16_as_ushort(__float2bfloat16_rn(__int_as_float(v[i]) + bias)));
-                    __syncwarp();
-#pragma unroll
-                    for (int j = 0; j < 2; ++j) {
-                        const int r = (lane >> 2) + 8 * j, f = w0 + (lane & 3) * 8;
+                        for (int i = 0; i < 16; i += 2) {
+                            const float z0 = __uint_as_float(v[h + i]) + bias, z1 = __uint_as_float(v[h + i + 1]) + bias;
+                            const float other = __shfl_xor_sync(0xffffffffu, hi ? z0 : z1, 8);
+                            sts_b16(at + i * 32, __bfloat16_as_ushort(__float2bfloat16_rn(gated<true>(hi ? other : z0, hi ? z1 : other, p.gate))));
+                        }
+                        __syncwarp();
+                        const int r = lane >> 1, f = w0 / 2 + (lane & 1) * 8;
                         if (c + r < cols && f < ldo)
-                            stg_128(reinterpret_cast<bf16*>(p.out) + (size_t)(t.row + c0 + c + r) * ldo + f, lds128(st + r * 64 + (lane & 3) * 16));
+                            stg_128(reinterpret_cast<bf16*>(p.out) + (size_t)(t.row + c0 + c + r) * ldo + f, lds128(st + r * 32 + (lane & 1) * 16));
+                    } else {
+#pragma unroll
+                        for (int i = 0; i < 16; ++i) sts_b16(st + i * 64 + lane * 2, __bfloat16_as_ushort(__float2bfloat16_rn(__uint_as_float(v[h + i]) + bias)));
+                        __syncwarp();
+#pragma unroll
+                        for (int j = 0; j < 2; ++j) {
+                            const int r = (lane >> 2) + 8 * j, f = w0 + (lane & 3) * 8;
+                            if (c + r < cols && f < ldo)
+                                stg_128(reinterpret_cast<bf16*>(p.out) + (size_t)(t.row + c0 + c + r) * ldo + f, lds128(st + r * 64 + (lane & 3) * 16));
+                        }
                     }
                 }
             }
