@@ -288,6 +288,7 @@ typedef struct {
     int* counts;               /* [E], or NULL */
     int* rank;                 /* [M][top] */
     int* slots;                /* [M][top] */
+    int* ticket;               /* decoder_moe_up_step: one word of workspace */
     const void* x;             /* [M][K] */
     void* sorted;              /* [M*top][K] */
     const void* w_up;          /* [E][2*ff][K] */

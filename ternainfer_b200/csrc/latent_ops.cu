@@ -222,7 +222,7 @@ static int moe_up_step(const MoeParams& p, int pdl, void* stream) {
 extern "C" int decoder_moe_up_step(const decoder_moe_args* a, int pdl, void* stream) {
     if (int rc = moe_check(a)) return rc;
     if (a->M > 8 || a->K % 8 || a->K > 12288 || a->gate.kind < 1 || a->gate.kind > 2) return bad(DECODER_BAD_SHAPE, "moe_up_step: M <= 8, K a multiple of 8 up to 12288");
-    if (!a->router || !a->router_bias || !a->chosen || !a->weight || !a->x || !a->w_up || !a->act || misaligned(a->router, 16) || misaligned(a->x, 16) ||
+    if (!a->router || !a->router_bias || !a->chosen || !a->weight || !a->ticket || !a->x || !a->w_up || !a->act || misaligned(a->router, 16) || misaligned(a->x, 16) ||
         misaligned(a->w_up, 16))
         return bad(DECODER_BAD_POINTER, "moe_up_step: null or misaligned pointer");
     const int rc = launch(router_step_kernel, dim3(a->M), 1024, (size_t)a->K * 2 + (size_t)a->E * 4, pdl, stream, 1, *a);
@@ -230,8 +230,8 @@ extern "C" int decoder_moe_up_step(const decoder_moe_args* a, int pdl, void* str
     // k-steps in flight: what leaves the last batch of a warp's share the fullest
     const int steps = ((a->K + 31) / 32 + kRowsWarps - 1) / kRowsWarps;
     const auto waste = [&](int n) { return (steps + n - 1) / n * n - steps; };
-    if (waste(6) <= waste(5) && waste(6) <= waste(4)) return moe_up_step<6>(*a, pdl, stream);
-    return waste(5) <= waste(4) ? moe_up_step<5>(*a, pdl, stream) : moe_up_step<4>(*a, pdl, stream);
+    if (waste(8) <= waste(6) && waste(8) <= waste(5)) return moe_up_step<8>(*a, pdl, stream);
+    return waste(6) <= waste(5) ? moe_up_step<6>(*a, pdl, stream) : moe_up_step<5>(*a, pdl, stream);
 }
 
 extern "C" int decoder_moe_down_step(const decoder_moe_args* a, int pdl, void* stream) {

@@ -180,6 +180,7 @@ static __global__ void __launch_bounds__(1024) router_step_kernel(const MoeParam
 #pragma unroll
     for (int i = 0; i < PRE; ++i) wv[i] = warp < p.E && lane + 32 * i < words ? ldg_stream_128(w + (size_t)warp * K + (lane + 32 * i) * 8) : make_uint4(0, 0, 0, 0);
     griddep_wait();
+    if (token == 0 && tid == 0) *p.ticket = 0;               // (the kernel after this one counts its work items here)
     for (int c = tid; c < words; c += blockDim.x) x_s[c] = __ldcg(reinterpret_cast<const uint4*>(p.x) + (size_t)token * words + c);
     __syncthreads();
     for (int e = warp; e < p.E; e += 32) {
@@ -214,18 +215,20 @@ static __global__ void __launch_bounds__(1024) router_step_kernel(const MoeParam
     }
 }
 
-// act[token * top + j][f].  Work items of 16 rows of gate and up of one chosen expert (8 activations), a contiguous share
-// per CTA; the weights' stream runs on across items, P k-steps per warp ahead.  The inputs lie in shared memory.
+// act[token * top + j][f].  Work items of 16 rows of gate and up of one chosen expert (8 activations), handed out as
+// the CTAs come for them (kernels before and after share the SMs unevenly); the weights' stream runs on across items, P k-steps per warp ahead.  The inputs lie in shared memory.
 template <int P>
 __global__ void __launch_bounds__(kRowsWarps * 32, 2) moe_up_step_kernel(const MoeParams p) {
     extern __shared__ __align__(16) uint8_t moe_up_smem[];   // inputs [M][K] bf16, rows 64 bytes longer
     __shared__ float part[2][kRowsWarps][16][9];
-    __shared__ int chosen[8 * kMoeMaxTop], list[8 * kMoeMaxTop];
+    __shared__ int chosen[8 * kMoeMaxTop], list[8 * kMoeMaxTop], drawn[2];
     griddep_launch_dependents();
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, q = lane & 3;
     const int K = p.K, steps = (K + 31) >> 5, top = p.top, blocks = p.ff / 8, xs = K * 2 + 64;
     const int s0 = steps * warp / kRowsWarps, s1 = steps * (warp + 1) / kRowsWarps;
     griddep_wait();
+    const auto draw = [&]() { return (int)gridDim.x + atomicAdd(p.ticket, 1); };
+    if (tid == 0) drawn[0] = draw();
     for (int i = tid; i < p.M * top; i += blockDim.x) chosen[i] = __ldcg(p.chosen + i);
     for (int i = tid; i < p.M * (K / 8); i += blockDim.x) {
         const int t = i / (K / 8), c = i - t * (K / 8);
@@ -233,41 +236,40 @@ __global__ void __launch_bounds__(kRowsWarps * 32, 2) moe_up_step_kernel(const M
     }
     __syncthreads();
     const int n = distinct_experts(chosen, p.M * top, p.E, list);
-    const int items = n * blocks, i0 = (int)((long long)items * blockIdx.x / gridDim.x), i1 = (int)((long long)items * (blockIdx.x + 1) / gridDim.x);
+    const int items = n * blocks;
     const bf16* w_up = reinterpret_cast<const bf16*>(p.w_up);
     const uint4 zero = make_uint4(0, 0, 0, 0);
-    const int batches = (s1 - s0 + P - 1) / P;               // per item
+    const int batches = max(1, (s1 - s0 + P - 1) / P);       // per item
     uint4 a[P], b[P];
     auto fetch = [&](int u, int item, int batch) {
         const int s = s0 + batch * P + u;
-        const bool in = item < i1 && s < s1 && 32 * s + q * 8 < K;
+        const bool in = item < items && s < s1 && 32 * s + q * 8 < K;
         const bf16* w = w_up;
         if (in) w += ((size_t)list[item / blocks] * 2 * p.ff + item % blocks * 16 + g) * K + 32 * s + q * 8;
         a[u] = in ? ldg_stream_128(w) : zero;
         b[u] = in ? ldg_stream_128(w + (size_t)8 * K) : zero;
     };
-    int next_item = i0, next_batch = 0;
-    auto advance = [&]() {
-        if (++next_batch >= batches) next_batch = 0, ++next_item;
-    };
-#pragma unroll
-    for (int u = 0; u < P; ++u) fetch(u, next_item, next_batch);
-    advance();
     const uint8_t* xrow = moe_up_smem + g * xs + q * 16;
-    for (int item = i0; item < i1; ++item) {
+    int item = (int)blockIdx.x, next = drawn[0];
+#pragma unroll
+    for (int u = 0; u < P; ++u) fetch(u, item, 0);
+    for (int turn = 0; item < items; ++turn) {
+        int after = 0;
+        if (tid == 0) after = draw();
         float acc[4] = {0.f, 0.f, 0.f, 0.f};
         for (int batch = 0; batch < batches; ++batch) {
+            const bool last = batch + 1 == batches;
 #pragma unroll
             for (int u = 0; u < P; ++u) {
                 const int s = s0 + batch * P + u;
                 const uint4 xv = g < p.M && s < s1 && 32 * s + q * 8 < K ? *reinterpret_cast<const uint4*>(xrow + 64 * s) : zero;
                 mma_bf16_16x8x16(acc, a[u].x, b[u].x, a[u].y, b[u].y, xv.x, xv.y);
                 mma_bf16_16x8x16(acc, a[u].z, b[u].z, a[u].w, b[u].w, xv.z, xv.w);
-                fetch(u, next_item, next_batch);
+                fetch(u, last ? next : item, last ? 0 : batch + 1);
             }
-            advance();
         }
-        float (*pt)[16][9] = part[(item - i0) & 1];          // written again two items later, behind a barrier
+        if (tid == 0) drawn[(turn + 1) & 1] = after;
+        float (*pt)[16][9] = part[turn & 1];          // written again two items later, behind a barrier
         pt[warp][g][2 * q] = acc[0], pt[warp][g][2 * q + 1] = acc[1];
         pt[warp][g + 8][2 * q] = acc[2], pt[warp][g + 8][2 * q + 1] = acc[3];
         __syncthreads();
@@ -282,6 +284,7 @@ __global__ void __launch_bounds__(kRowsWarps * 32, 2) moe_up_step_kernel(const M
                 if (chosen[t * top + j] == e) pair = t * top + j;
             if (r < 8 && pair >= 0) reinterpret_cast<bf16*>(p.act)[(size_t)pair * p.ff + item % blocks * 8 + r] = from_f<bf16>(gated(v, up, p.gate));
         }
+        item = next, next = drawn[(turn + 1) & 1];
     }
 }
 

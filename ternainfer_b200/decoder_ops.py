@@ -384,7 +384,9 @@ def expert_step(x, router, router_bias, top: int, w_up, gate: Gate, step: bool =
     E, ff = w_up.shape[0], w_up.shape[1] // 2
     chosen, weight = _choices(M, top, x.device)
     act = torch.empty((M, top, ff), dtype=x.dtype, device=x.device)
-    a = _moe(M, E, top, K, ff, gate=gate, router=router, router_bias=router_bias, chosen=chosen, weight=weight, x=x, w_up=w_up, act=act)
+    ticket = torch.empty((1,), dtype=torch.int32, device=x.device)
+    a = _moe(M, E, top, K, ff, gate=gate, router=router, router_bias=router_bias, chosen=chosen, weight=weight, ticket=ticket, x=x, w_up=w_up,
+             act=act)
     _dtype(x)
     check(load_decoder_library().decoder_moe_up_step(ctypes.byref(a), int(step), _stream()))
     return act, chosen, weight

@@ -61,7 +61,7 @@ RotateArgs = _struct("RotateArgs", ["p src dst trig pos", "i B T H rot dims", "l
 AbsorbArgs = _struct("AbsorbArgs", ["p q w_uk_t qa trig pos", "i B T H dim rot dims R r_at ld"])
 LatentAttnArgs = _struct("LatentAttnArgs", ["p qa cache sink pos out w_uv part ml y", "i B T H R ld vdim slots splits cluster", "f scale"])
 LatentPromptArgs = _struct("LatentPromptArgs", ["p q kv cache sink y", "i B T H dim rot vdim slots ld r_at start off_v", "l ld_kv", "f scale"])
-MoeArgs = _struct("MoeArgs", ["p logits router router_bias chosen weight counts rank slots x sorted w_up act w_down w_rest rest bias out",
+MoeArgs = _struct("MoeArgs", ["p logits router router_bias chosen weight counts rank slots ticket x sorted w_up act w_down w_rest rest bias out",
                               "i M E top K ff D K_rest", "g gate"])
 GroupGemmArgs = _struct("GroupGemmArgs", ["p a w bias counts out", "i rows groups N K", "g gate"])
 
