@@ -1342,16 +1342,18 @@ def sidirax_kernels(torch, size, args):
         put(f"{tag}/dense_down_and_mixer_out", [lambda w=w, o=wo[i % 8]: ops.down_step(act, w, db, rest=a, w_rest=o, step=True) for i, w in enumerate(ws)],
             nb, 2.0 * B * (ff + n) * width)
         del ws
-        xs = [rnd(B, width) for _ in range(20)]
-        used, acts = [], []
-        for x in xs:
-            acts.append(ops.expert_step(x, rw, rb, top, up[0], silu))
-            used.append(acts[-1][1].unique().numel())
-        used = sum(used) / len(used)
-        put(f"{tag}/router_and_expert_up", [lambda x=x, w=up[i % 2]: ops.expert_step(x, rw, rb, top, w, silu, True) for i, x in enumerate(xs)],
-            2.0 * (used * 2 * fe * width + E * width + B * (width + top * fe)), 4.0 * B * top * fe * width)
-        put(f"{tag}/expert_down_and_mixer_out", [lambda t=t, w=down[i % 2], o=wo[i % 8]: ops.down_step(t[0], w, None, t[1], t[2], a, o, True)
-                                                 for i, t in enumerate(acts)],
+        routes, acts = [ops.Routing(rnd(B, width), rw, rb, top) for _ in range(20)], []
+        tickets = torch.zeros(20, dtype=torch.int32, device=dev)           # zeroed once per list; in the model, by the projection before
+        for i, r in enumerate(routes):
+            r.logits.copy_(ops.linear_fp32(r.x, rw))
+            r.ticket = tickets[i:i + 1]
+            acts.append(ops.expert_step(r, up[0], silu))
+        used = sum(r.chosen.unique().numel() for r in routes) / 20
+        put(f"{tag}/routing_and_expert_up", [lambda i=i, r=r: (tickets.zero_() if i == 0 else None, ops.expert_step(r, up[i % 2], silu, True))
+                                             for i, r in enumerate(routes)],
+            2.0 * (used * 2 * fe * width + B * (width + top * fe)), 4.0 * B * top * fe * width)
+        put(f"{tag}/expert_down_and_mixer_out", [lambda t=t, r=r, w=down[i % 2], o=wo[i % 8]: ops.down_step(t, w, None, r, a, o, True)
+                                                 for i, (t, r) in enumerate(zip(acts, routes))],
             2.0 * (used * fe * width + width * n + B * (top * fe + n + width)), 2.0 * B * (top * fe + n) * width)
         xr, y, prev = f32(B, 1, width), rnd(B, width), rnd(B, width)
         put(f"{tag}/residual_norm", [lambda: ops.hyper_norm(xr, w1, eps, bf, y=y, step=True)] * 20, 12.0 * B * width)

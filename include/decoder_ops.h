@@ -87,13 +87,18 @@ typedef struct {
 
 /* out[m][n] = act(sum_k w[n][k] x[m][k] + bias[n]), bf16 in, M <= 8, K a multiple of 8; out_fp32: fp32 instead of bf16
  * results.  seg_rows > 0: rows [s * seg_rows, (s + 1) * seg_rows) of w (the last of n_seg segments: all further rows)
- * read x + s * M * K.  gate.kind > 0: w and bias hold blocks of 8 gate and 8 up rows, out is [M][N / 2]. */
+ * read x + s * M * K.  gate.kind > 0: w and bias hold blocks of 8 gate and 8 up rows, out is [M][N / 2].  N2 > 0: in the
+ * same launch out2 = w2 x2, fp32; zero: a word to be set to 0 with it (decoder_moe_up_step's ticket). */
 typedef struct {
     const void* x;             /* [n_seg][M][K] */
     const void* w;             /* [N][K] */
     const float* bias;         /* [N], or NULL */
     void* out;                 /* [M][N] */
-    int M, N, K, relu2, seg_rows, n_seg;
+    const void* x2;            /* [M][K] */
+    const void* w2;            /* [N2][K] */
+    float* out2;               /* [M][N2] */
+    int* zero;                 /* or NULL */
+    int M, N, K, relu2, seg_rows, n_seg, N2;
     decoder_gate gate;
 } decoder_linear_args;
 int decoder_rows_linear(const decoder_linear_args* a, int out_fp32, int pdl, void* stream);
@@ -277,11 +282,10 @@ int decoder_latent_prompt(const decoder_latent_prompt_args* a, void* stream);
  * decoder_moe_route: chosen experts and weights; with counts (zeroed by the caller) also every choice's rank among its
  *   expert's, then the rows of x sorted by expert, slots[token][j] saying where a choice's row went (bf16, K % 8 = 0).
  * decoder_moe_plain: any type and size, chosen and weight given: act, and out [M*top][D] not weighted.
- * decoder_moe_up_step: bf16, M <= 8, K a multiple of 8 up to 12288: routing (router instead of logits) and activations.
+ * decoder_moe_up_step: bf16, M <= 8, K a multiple of 8 up to 12288: routing and activations; ticket must be 0 before.
  * decoder_moe_down_step: bf16, M <= 8: out [M][D] = weighted sum + w_rest rest + bias.  Dense: weight NULL, E = top = 1. */
 typedef struct {
     const float* logits;       /* [M][E], without bias */
-    const void* router;        /* [E][K] */
     const float* router_bias;  /* [E] */
     int* chosen;               /* [M][top] */
     float* weight;             /* [M][top] */

@@ -62,7 +62,8 @@ extern "C" int decoder_rows_linear(const decoder_linear_args* a, int out_fp32, i
     if (a->seg_rows < 0 || a->seg_rows % 16 || (a->seg_rows && a->n_seg < 1)) return bad(DECODER_BAD_SHAPE, "rows_linear: segments of 16 rows");
     if (a->gate.kind < 0 || a->gate.kind > 2 || (a->gate.kind && a->N % 16)) return bad(DECODER_BAD_SHAPE, "rows_linear: gated rows come in blocks of 16");
     if (!a->x || !a->w || !a->out || misaligned(a->x, 16) || misaligned(a->w, 16)) return bad(DECODER_BAD_POINTER, "rows_linear: null or misaligned pointer");
-    const dim3 grid((a->N + 15) / 16);
+    if (a->N2 < 0 || (a->N2 && (!a->w2 || !a->x2 || !a->out2 || misaligned(a->w2, 16) || misaligned(a->x2, 16)))) return bad(DECODER_BAD_POINTER, "rows_linear: second product");
+    const dim3 grid((a->N + 15) / 16 + (a->N2 + 15) / 16);
     return out_fp32 ? launch(rows_linear_kernel<float>, grid, kRowsWarps * 32, 0, pdl, stream, 1, *a)
                     : launch(rows_linear_kernel<bf16>, grid, kRowsWarps * 32, 0, pdl, stream, 1, *a);
 }

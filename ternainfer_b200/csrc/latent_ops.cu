@@ -216,17 +216,15 @@ extern "C" int decoder_moe_plain(const decoder_moe_args* a, int dtype, int pdl, 
 template <int P>
 static int moe_up_step(const MoeParams& p, int pdl, void* stream) {
     const int items = p.ff / 8 * std::min(p.E, p.M * p.top);
-    return launch(moe_up_step_kernel<P>, dim3(std::min(items, 2 * sm_count())), kRowsWarps * 32, (size_t)p.M * (p.K * 2 + 64), pdl, stream, 1, p);
+    return launch(moe_up_step_kernel<P>, dim3(std::min(items, 2 * sm_count())), kRowsWarps * 32, (size_t)p.M * (p.K * 2 + 64 + p.E * 4), pdl, stream, 1, p);
 }
 
 extern "C" int decoder_moe_up_step(const decoder_moe_args* a, int pdl, void* stream) {
     if (int rc = moe_check(a)) return rc;
     if (a->M > 8 || a->K % 8 || a->K > 12288 || a->gate.kind < 1 || a->gate.kind > 2) return bad(DECODER_BAD_SHAPE, "moe_up_step: M <= 8, K a multiple of 8 up to 12288");
-    if (!a->router || !a->router_bias || !a->chosen || !a->weight || !a->ticket || !a->x || !a->w_up || !a->act || misaligned(a->router, 16) || misaligned(a->x, 16) ||
+    if (!a->logits || !a->router_bias || !a->chosen || !a->weight || !a->ticket || !a->x || !a->w_up || !a->act || misaligned(a->x, 16) ||
         misaligned(a->w_up, 16))
         return bad(DECODER_BAD_POINTER, "moe_up_step: null or misaligned pointer");
-    const int rc = launch(router_step_kernel, dim3(a->M), 1024, (size_t)a->K * 2 + (size_t)a->E * 4, pdl, stream, 1, *a);
-    if (rc) return rc;
     // k-steps in flight: what leaves the last batch of a warp's share the fullest
     const int steps = ((a->K + 31) / 32 + kRowsWarps - 1) / kRowsWarps;
     const auto waste = [&](int n) { return (steps + n - 1) / n * n - steps; };

@@ -5,8 +5,8 @@
 //
 // Weights: gate and up rows in blocks of eight in one matrix [E][2 * ff][K] (gate.cuh), down [E][D][ff]; ff padded to a
 // multiple of 8.  Prompts (bf16): rows are sorted by expert and go through the grouped GEMM (group_gemm_tc.cuh); the
-// residual kernel adds the weighted results (hyper.cuh).  Up to eight tokens: one launch routes, one makes the
-// activations, expert by expert, so that an expert's weights are read once for all its tokens; a third one sums the
+// residual kernel adds the weighted results (hyper.cuh).  Up to eight tokens: one launch routes and makes the
+// activations, expert by expert, so that an expert's weights are read once for all its tokens; a second one sums the
 // down projections of all experts, and the mixer's output projection with them, without leaving the registers.
 // Other types and sizes: one warp per output.
 #pragma once
@@ -167,59 +167,11 @@ __device__ __forceinline__ int distinct_experts(const int* chosen, int n, int E,
     return count;
 }
 
-// Router of up to eight tokens: one CTA per token makes the logits, one warp per expert in turn, and chooses.
-static __global__ void __launch_bounds__(1024) router_step_kernel(const MoeParams p) {
-    extern __shared__ __align__(16) uint8_t router_smem[];   // the token's input [K] bf16, logits [E]
-    griddep_launch_dependents();
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, token = blockIdx.x, K = p.K, words = K / 8;
-    const bf16* w = reinterpret_cast<const bf16*>(p.router);
-    uint4* x_s = reinterpret_cast<uint4*>(router_smem);
-    float* z_s = reinterpret_cast<float*>(router_smem + (size_t)words * 16);
-    constexpr int PRE = 8;                                   // words of the warp's first expert that are under way before the wait
-    uint4 wv[PRE];
-#pragma unroll
-    for (int i = 0; i < PRE; ++i) wv[i] = warp < p.E && lane + 32 * i < words ? ldg_stream_128(w + (size_t)warp * K + (lane + 32 * i) * 8) : make_uint4(0, 0, 0, 0);
-    griddep_wait();
-    if (token == 0 && tid == 0) *p.ticket = 0;               // (the kernel after this one counts its work items here)
-    for (int c = tid; c < words; c += blockDim.x) x_s[c] = __ldcg(reinterpret_cast<const uint4*>(p.x) + (size_t)token * words + c);
-    __syncthreads();
-    for (int e = warp; e < p.E; e += 32) {
-        float z = 0.f;
-        for (int c0 = 0; c0 < words; c0 += 32 * PRE) {
-            if (e != warp || c0)
-#pragma unroll
-                for (int i = 0; i < PRE; ++i) {
-                    const int c = c0 + lane + 32 * i;
-                    wv[i] = c < words ? ldg_stream_128(w + (size_t)e * K + c * 8) : make_uint4(0, 0, 0, 0);
-                }
-#pragma unroll
-            for (int i = 0; i < PRE; ++i) {
-                const int c = c0 + lane + 32 * i;
-                if (c < words) {
-                    float a[8], b[8];
-                    unpack8(wv[i], a), unpack8(x_s[c], b);
-#pragma unroll
-                    for (int j = 0; j < 8; ++j) z = fmaf(a[j], b[j], z);
-                }
-            }
-        }
-        z = warp_sum(z);
-        if (lane == 0) z_s[e] = z + p.router_bias[e];
-    }
-    __syncthreads();
-    if (warp == 0) {
-        int e;
-        float wt;
-        choose(z_s, p.E, p.top, lane, e, wt);
-        if (lane < p.top) p.chosen[token * p.top + lane] = e, p.weight[token * p.top + lane] = wt;
-    }
-}
-
-// act[token * top + j][f].  Work items of 16 rows of gate and up of one chosen expert (8 activations), handed out as
+// Routing, then act[token * top + j][f].  Every CTA makes the choices for itself.  Work items of 16 rows of gate and up of one chosen expert (8 activations), handed out as
 // the CTAs come for them (kernels before and after share the SMs unevenly); the weights' stream runs on across items, P k-steps per warp ahead.  The inputs lie in shared memory.
 template <int P>
 __global__ void __launch_bounds__(kRowsWarps * 32, 2) moe_up_step_kernel(const MoeParams p) {
-    extern __shared__ __align__(16) uint8_t moe_up_smem[];   // inputs [M][K] bf16, rows 64 bytes longer
+    extern __shared__ __align__(16) uint8_t moe_up_smem[];   // inputs [M][K] bf16, rows 64 bytes longer; logits [M][E]
     __shared__ float part[2][kRowsWarps][16][9];
     __shared__ int chosen[8 * kMoeMaxTop], list[8 * kMoeMaxTop], drawn[2];
     griddep_launch_dependents();
@@ -229,7 +181,18 @@ __global__ void __launch_bounds__(kRowsWarps * 32, 2) moe_up_step_kernel(const M
     griddep_wait();
     const auto draw = [&]() { return (int)gridDim.x + atomicAdd(p.ticket, 1); };
     if (tid == 0) drawn[0] = draw();
-    for (int i = tid; i < p.M * top; i += blockDim.x) chosen[i] = __ldcg(p.chosen + i);
+    if (warp < p.M) {
+        float* z = reinterpret_cast<float*>(moe_up_smem + p.M * xs) + warp * p.E;
+        for (int i = lane; i < p.E; i += 32) z[i] = __ldcg(p.logits + (size_t)warp * p.E + i) + p.router_bias[i];
+        __syncwarp();
+        int e;
+        float w;
+        choose(z, p.E, top, lane, e, w);
+        if (lane < top) {
+            chosen[warp * top + lane] = e;
+            if (blockIdx.x == 0) p.chosen[warp * top + lane] = e, p.weight[warp * top + lane] = w;
+        }
+    }
     for (int i = tid; i < p.M * (K / 8); i += blockDim.x) {
         const int t = i / (K / 8), c = i - t * (K / 8);
         *reinterpret_cast<uint4*>(moe_up_smem + t * xs + c * 16) = __ldcg(reinterpret_cast<const uint4*>(p.x) + i);

@@ -7,7 +7,8 @@
 // previous kernel of the stream, so the weights' latency runs underneath its tail.  The rows of x are the
 // MMA's N = 8 and come from L2.  Warp partials meet in shared memory in a fixed order.
 // W may consist of segments of rows with an input each (projections of one token's differently mixed inputs in one
-// launch).  Gated feed-forwards: W holds blocks of 8 gate and 8 up rows, so a CTA makes 8 activations.
+// launch).  A second product of the same row length (a router's logits) may ride along in CTAs of its own, with fp32
+// results.  Gated feed-forwards: W holds blocks of 8 gate and 8 up rows, so a CTA makes 8 activations.
 #pragma once
 #include "decoder_common.cuh"
 #include "decoder_ops.h"
@@ -28,14 +29,16 @@ __global__ void __launch_bounds__(kRowsWarps * 32, 2) rows_linear_kernel(const R
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int g = lane >> 2, q = lane & 3;
     const int K = p.K, steps = (K + 31) >> 5;
-    const int n0 = blockIdx.x * 16;
+    const int blocks = (p.N + 15) >> 4;
+    const bool side = (int)blockIdx.x >= blocks;
+    const int n0 = ((int)blockIdx.x - (side ? blocks : 0)) * 16, N = side ? p.N2 : p.N;
     const int s0 = steps * warp / kRowsWarps, s1 = steps * (warp + 1) / kRowsWarps;
-    const bool ok0 = n0 + g < p.N, ok1 = n0 + g + 8 < p.N;
-    const bf16* w = reinterpret_cast<const bf16*>(p.w);
+    const bool ok0 = n0 + g < N, ok1 = n0 + g + 8 < N;
+    const bf16* w = reinterpret_cast<const bf16*>(side ? p.w2 : p.w);
     const bf16* w0 = w + (size_t)(ok0 ? n0 + g : 0) * K + q * 8;
     const bf16* w1 = w + (size_t)(ok1 ? n0 + g + 8 : 0) * K + q * 8;
-    const int seg = p.seg_rows > 0 ? min(n0 / p.seg_rows, p.n_seg - 1) : 0;
-    const bf16* x = reinterpret_cast<const bf16*>(p.x) + (size_t)seg * p.M * K + (size_t)(g < p.M ? g : 0) * K + q * 8;
+    const int seg = !side && p.seg_rows > 0 ? min(n0 / p.seg_rows, p.n_seg - 1) : 0;
+    const bf16* x = reinterpret_cast<const bf16*>(side ? p.x2 : p.x) + (size_t)seg * p.M * K + (size_t)(g < p.M ? g : 0) * K + q * 8;
     const bool xok = g < p.M;
     const uint4 zero = make_uint4(0, 0, 0, 0);
     uint4 a[kRowsPre], b[kRowsPre];
@@ -68,7 +71,12 @@ __global__ void __launch_bounds__(kRowsWarps * 32, 2) rows_linear_kernel(const R
         float v = 0.f;
 #pragma unroll
         for (int i = 0; i < kRowsWarps; ++i) v += part[i][r][t];
-        const bool live = t < p.M && n0 + r < p.N;
+        const bool live = t < p.M && n0 + r < N;
+        if (side) {
+            if (live) p.out2[(size_t)t * N + n0 + r] = v;
+            if (p.zero && n0 == 0 && tid == 0) *p.zero = 0;
+            return;
+        }
         if (p.bias && n0 + r < p.N) v += p.bias[n0 + r];
         if (p.gate.kind) {
             const float up = __shfl_down_sync(0xffffffffu, v, 8);

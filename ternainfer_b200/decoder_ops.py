@@ -98,17 +98,32 @@ def few_rows(x: torch.Tensor) -> bool:
     return x.dtype == torch.bfloat16 and x.shape[-2] <= ROWS and x.shape[-1] % 8 == 0
 
 
+class Routing:
+    """What routes up to 8 bf16 rows [M, K] among the experts of a router [E, K]: the rows, the logits that a linear before
+    makes beside its own product (``rows_linear``), the choices and weights that ``expert_step`` makes of them."""
+
+    def __init__(self, x, router, bias, top: int):
+        M = x.shape[0]
+        self.x, self.router, self.bias, self.top = x, router, bias, top
+        self.logits = torch.empty((M, router.shape[0]), dtype=torch.float32, device=x.device)
+        self.chosen, self.weight = _choices(M, top, x.device)
+        self.ticket = torch.empty((1,), dtype=torch.int32, device=x.device)
+
+
 def rows_linear(x, weight, bias=None, gate: Gate = NO_GATE, relu2: bool = False, fp32: bool = False, seg_rows: int = 0,
-                step: bool = False) -> torch.Tensor:
+                step: bool = False, route: Optional[Routing] = None) -> torch.Tensor:
     """The streaming linear for up to 8 bf16 rows.  x [M, K], or [segments, M, K] when every ``seg_rows`` rows of the
     weight (the last segment: all that are left) read their own input.  ``gate``: weight and bias (fp32) hold blocks of
-    8 gate and 8 up rows."""
+    8 gate and 8 up rows.  ``route``: its logits are made in the same launch."""
     M, K = x.shape[-2:]
     N = weight.shape[0]
     _dtype(x)
     out = torch.empty((M, N // 2 if gate.kind else N), dtype=torch.float32 if fp32 else x.dtype, device=x.device)
-    a = LinearArgs(x.data_ptr(), weight.data_ptr(), _ptr(bias), out.data_ptr(), M, N, K, int(relu2), seg_rows,
-                   x.shape[0] if seg_rows else 0, gate)
+    a = LinearArgs(x=x.data_ptr(), w=weight.data_ptr(), bias=_ptr(bias), out=out.data_ptr(), M=M, N=N, K=K, relu2=int(relu2), seg_rows=seg_rows,
+                   n_seg=x.shape[0] if seg_rows else 0, gate=gate)
+    if route is not None:
+        a.x2, a.w2, a.out2, a.zero, a.N2 = (route.x.data_ptr(), route.router.data_ptr(), route.logits.data_ptr(), route.ticket.data_ptr(),
+                                            route.router.shape[0])
     check(load_decoder_library().decoder_rows_linear(ctypes.byref(a), int(fp32), int(step), _stream()))
     return out
 
@@ -378,29 +393,25 @@ def _choices(M: int, top: int, device):
     return torch.empty((M, top), dtype=torch.int32, device=device), torch.empty((M, top), dtype=torch.float32, device=device)
 
 
-def expert_step(x, router, router_bias, top: int, w_up, gate: Gate, step: bool = False):
-    """Up to 8 bf16 rows: routing and the chosen experts' activations [M, top, ff], with the choices [M, top] and weights."""
-    M, K = x.shape
+def expert_step(route: Routing, w_up, gate: Gate, step: bool = False) -> torch.Tensor:
+    """Choices and weights of the routed rows, and the chosen experts' activations [M, top, ff]."""
+    M, K = route.x.shape
     E, ff = w_up.shape[0], w_up.shape[1] // 2
-    chosen, weight = _choices(M, top, x.device)
-    act = torch.empty((M, top, ff), dtype=x.dtype, device=x.device)
-    ticket = torch.empty((1,), dtype=torch.int32, device=x.device)
-    a = _moe(M, E, top, K, ff, gate=gate, router=router, router_bias=router_bias, chosen=chosen, weight=weight, ticket=ticket, x=x, w_up=w_up,
-             act=act)
-    _dtype(x)
+    act = torch.empty((M, route.top, ff), dtype=route.x.dtype, device=route.x.device)
+    a = _moe(M, E, route.top, K, ff, gate=gate, logits=route.logits, router_bias=route.bias, chosen=route.chosen, weight=route.weight,
+             ticket=route.ticket, x=route.x, w_up=w_up, act=act)
+    _dtype(act)
     check(load_decoder_library().decoder_moe_up_step(ctypes.byref(a), int(step), _stream()))
-    return act, chosen, weight
+    return act
 
 
-def down_step(act, w_down, bias=None, chosen=None, weight=None, rest=None, w_rest=None, step: bool = False) -> torch.Tensor:
+def down_step(act, w_down, bias=None, route: Optional[Routing] = None, rest=None, w_rest=None, step: bool = False) -> torch.Tensor:
     """Up to 8 bf16 rows, one launch: W_down act [M, ff], or the weighted sum over chosen experts (act [M, top, ff]), plus
     W_rest rest and a bias (fp32)."""
     M, ff = act.shape[0], act.shape[-1]
-    routed = weight is not None
-    E, D = (w_down.shape[0], w_down.shape[1]) if routed else (1, w_down.shape[0])
-    out = torch.empty((M, D), dtype=act.dtype, device=act.device)
-    a = _moe(M, E, act.shape[1] if routed else 1, 8, ff, D, K_rest=0 if rest is None else rest.shape[1], chosen=chosen, weight=weight, act=act,
-             w_down=w_down, w_rest=w_rest, rest=rest, bias=bias, out=out)
+    out = torch.empty((M, w_down.shape[-2]), dtype=act.dtype, device=act.device)
+    a = _moe(M, w_down.shape[0] if route else 1, route.top if route else 1, 8, ff, w_down.shape[-2], K_rest=0 if rest is None else rest.shape[1],
+             chosen=route and route.chosen, weight=route and route.weight, act=act, w_down=w_down, w_rest=w_rest, rest=rest, bias=bias, out=out)
     _dtype(act)
     check(load_decoder_library().decoder_moe_down_step(ctypes.byref(a), int(step), _stream()))
     return out

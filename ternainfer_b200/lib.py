@@ -49,7 +49,7 @@ EmbedArgs = _struct("EmbedArgs", ["p tokens pos prev embed bigram x", "l mul_pre
 HyperArgs = _struct("HyperArgs", ["p x y mix out in_ w rows h y2 slots slot_w mu prev mixed pos", "f m w_offset eps",
                                   "i D S n_rows top n_mu"])
 ShiftArgs = _struct("ShiftArgs", ["p h prev mu mixed pos", "i B T D n_mu"])
-LinearArgs = _struct("LinearArgs", ["p x w bias out", "i M N K relu2 seg_rows n_seg", "g gate"])
+LinearArgs = _struct("LinearArgs", ["p x w bias out x2 w2 out2 zero", "i M N K relu2 seg_rows n_seg N2", "g gate"])
 DeltaArgs = _struct("DeltaArgs", ["p proj zw w2 w0 a_bias norm pos state o y", "i B T H dk dv rank", "l ld",
                                   "i off_r off_k off_v off_a off_g off_w1", "f eps"])
 AttnArgs = _struct("AttnArgs", ["p proj ck cv q_norm k_norm bias slope pos y", "i B T H G dim vdim", "l ld",
@@ -61,7 +61,7 @@ RotateArgs = _struct("RotateArgs", ["p src dst trig pos", "i B T H rot dims", "l
 AbsorbArgs = _struct("AbsorbArgs", ["p q w_uk_t qa trig pos", "i B T H dim rot dims R r_at ld"])
 LatentAttnArgs = _struct("LatentAttnArgs", ["p qa cache sink pos out w_uv part ml y", "i B T H R ld vdim slots splits cluster", "f scale"])
 LatentPromptArgs = _struct("LatentPromptArgs", ["p q kv cache sink y", "i B T H dim rot vdim slots ld r_at start off_v", "l ld_kv", "f scale"])
-MoeArgs = _struct("MoeArgs", ["p logits router router_bias chosen weight counts rank slots ticket x sorted w_up act w_down w_rest rest bias out",
+MoeArgs = _struct("MoeArgs", ["p logits router_bias chosen weight counts rank slots ticket x sorted w_up act w_down w_rest rest bias out",
                               "i M E top K ff D K_rest", "g gate"])
 GroupGemmArgs = _struct("GroupGemmArgs", ["p a w bias counts out", "i rows groups N K", "g gate"])
 

@@ -39,8 +39,8 @@ class FusedProjection(nn.Module):
         weight[:at] = torch.cat([w.to(dtype) for w in parts.values()])
         self.weight = nn.Parameter(weight, requires_grad=False)
 
-    def forward(self, h, step: bool = False):
-        return ops.linear(h, self.weight, step=step)
+    def forward(self, h, step: bool = False, route=None):
+        return ops.linear(h, self.weight, step=step) if route is None else ops.rows_linear(h, self.weight, step=step, route=route)
 
 
 def _param(t: torch.Tensor, dtype=torch.float32):
@@ -127,11 +127,12 @@ class WkvMixer(nn.Module):
         return (torch.zeros((batch, self.heads, self.dim, self.dim), device=device, dtype=torch.float32),
                 torch.zeros((batch, self.mu.shape[1]), device=device, dtype=dtype))
 
-    def forward(self, mixed, cache, pos, T: int, step: bool = False):
-        """mixed [5 or more, B*T, D]: the inputs of ``MIXED`` (``ops.token_shift``, ``ops.hyper_norm``)."""
+    def forward(self, mixed, cache, pos, T: int, step: bool = False, route: Optional[ops.Routing] = None):
+        """mixed [5 or more, B*T, D]: the inputs of ``MIXED`` (``ops.token_shift``, ``ops.hyper_norm``).  route: logits to be
+        made beside the first projection."""
         n, s = self.heads * self.dim, self.seg
         if ops.few_rows(mixed):
-            z = ops.rows_linear(mixed[:5], self.weight, seg_rows=s, step=step)
+            z = ops.rows_linear(mixed[:5], self.weight, seg_rows=s, step=step, route=route)
             r, k, v, g, t1 = (z[:, i * s:] for i in range(5))
         else:
             r, k, v, g = torch.bmm(mixed[:4], self.weight[:4 * s].view(4, s, -1).transpose(1, 2))
@@ -202,10 +203,11 @@ class LatentAttention(nn.Module):
     def make_cache(self, batch: int, max_seq_len: int, device, dtype):
         return latent_cache(batch, max_seq_len, self.ld, device, dtype) if self.own else ()
 
-    def forward(self, h, cache, pos, T: int, start: Optional[int] = None, step: bool = False):
-        """cache: this layer's, or that of the layer whose latent it reads, already holding these tokens."""
+    def forward(self, h, cache, pos, T: int, start: Optional[int] = None, step: bool = False, route: Optional[ops.Routing] = None):
+        """cache: this layer's, or that of the layer whose latent it reads, already holding these tokens.  route: logits to be
+        made beside the first projection."""
         H, d, r, dv = self.heads, self.dim, self.rot_dim, self.vdim
-        z, at = self.proj(h, step), self.proj.offsets
+        z, at = self.proj(h, step, route), self.proj.offsets
         own = dict(cache=cache, off_kv=at["dkv"], kv_norm=self.kv_norm, r_at=self.r_at, rot=r, trig=self.trig) if self.own else {}
         q = ops.linear(ops.latent_prep(z, at["dq"], self.q_norm, pos, T, self.eps, step=step, **own), self.uq, step=step)
         bf16, w_uv = q.dtype == torch.bfloat16, self.ukv[H * d:]
@@ -266,11 +268,17 @@ class ExpertFeedForward(nn.Module):
         self.router, self.router_bias = _param(w["router"], dtype), _param(w["router.b"])
         self.up, self.down = _param(gated_rows(stack("gate"), stack("up")), dtype), _param(_pad_columns(stack("down")), dtype)
 
-    def forward(self, h, rest=None, step: bool = False) -> dict:
+    def routing(self, h) -> Optional[ops.Routing]:
+        """For few rows: the routing whose logits the mixer's first projection makes in passing; otherwise None."""
+        return ops.Routing(h, self.router, self.router_bias, self.top) if ops.few_rows(h) and h.shape[1] <= 12288 else None
+
+    def forward(self, h, rest=None, step: bool = False, route: Optional[ops.Routing] = None) -> dict:
         a, w_rest = rest or (None, None)
-        if ops.few_rows(h) and h.shape[1] <= 12288 and (a is None or a.shape[1] % 8 == 0):
-            act, chosen, weight = ops.expert_step(h, self.router, self.router_bias, self.top, self.up, self.gate, step)
-            return {"y": ops.down_step(act, self.down, None, chosen, weight, a, w_rest, step)}
+        if route is not None:
+            act = ops.expert_step(route, self.up, self.gate, step)
+            if a is None or a.shape[1] % 8 == 0:
+                return {"y": ops.down_step(act, self.down, None, route, a, w_rest, step)}
+            return {"y": ops.linear(a, w_rest, step=step), "y2": ops.down_step(act, self.down, None, route, step=step)}
         out, slots, weight = ops.expert_rows(h, self.router, self.router_bias, self.top, self.up, self.down, self.gate)
         y = torch.zeros_like(h) if a is None else ops.linear(a, w_rest, step=step)
         return {"y": y, "y2": out, "slots": slots, "slot_w": weight}

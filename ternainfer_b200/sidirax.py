@@ -238,8 +238,13 @@ class Sidirax(nn.Module):
                 mixed = ops.token_shift(h, layer.mixer.mu, held[1], pos, T) if layer.recurrent else None
             if on_layer is not None and i:
                 on_layer(i - 1, x[:, 0].clone())
-            y = layer.mixer(mixed, held, pos, T, step) if layer.recurrent else layer.mixer(h, held, pos, T, start, step)
-            write = {"y": ops.linear(y, layer.mixer.o, step=step)} if layer.ff is None else layer.ff(h, (y, layer.mixer.o), step)
+            route = layer.ff.routing(h) if isinstance(layer.ff, ExpertFeedForward) else None
+            y = layer.mixer(mixed, held, pos, T, step, route) if layer.recurrent else layer.mixer(h, held, pos, T, start, step, route)
+            rest = (y, layer.mixer.o)
+            if layer.ff is None:
+                write = {"y": ops.linear(*rest, step=step)}
+            else:
+                write = layer.ff(h, rest, step) if route is None else layer.ff(h, rest, step, route)
         if on_layer is not None:
             ops.hyper_norm(x, self.norm, a.eps, self.dtype, **write)
             write = {}

@@ -449,6 +449,19 @@ def ff_module(cfg, w, dtype):
     return ExpertFeedForward(cfg["router"]["experts"], cfg["router"]["top"], ops.silu_gate(), w, dtype).cuda()
 
 
+def run_ff(f, h, rest=None, step=False):
+    """The feed-forward as the model calls it: few rows are routed by logits that some projection makes in passing."""
+    from ternainfer_b200 import decoder_ops as ops
+    h = h.cuda()
+    route = f.routing(h) if hasattr(f, "routing") else None
+    if route is None:
+        return f(h, rest, step)
+    w = torch.randn((24, h.shape[1]), generator=torch.Generator().manual_seed(0)).to(h.dtype)
+    y = ops.rows_linear(h, w.cuda(), step=step, route=route)
+    assert rel_rms(y, h.double().cpu() @ w.double().T) < 5e-3
+    return f(h, rest, step, route)
+
+
 def ff_total(out):
     """What the residual would receive."""
     y = out["y"].double()
@@ -471,9 +484,11 @@ def test_feed_forwards(dec, cfg, dtype):
         h = (1.5 * torch.randn((M, D), generator=g)).to(dtype)
         a, wo = torch.randn((M, 40), generator=g).to(dtype), (torch.randn((D, 40), generator=g) / 40 ** 0.5).to(dtype)
         want = o.feed_forward(h.double(), {k: v.double() for k, v in w.items()}, "", cfg)
-        assert rel_rms(ff_total(f(h.cuda())), want) < TOL[dtype], (D, M)
+        assert rel_rms(ff_total(run_ff(f, h)), want) < TOL[dtype], (D, M)
         both = want + a.double() @ wo.double().T
-        assert rel_rms(ff_total(f(h.cuda(), (a.cuda(), wo.cuda()), step=M <= 8)), both) < TOL[dtype], (D, M)
+        assert rel_rms(ff_total(run_ff(f, h, (a.cuda(), wo.cuda()), step=M <= 8)), both) < TOL[dtype], (D, M)
+        odd = want + a[:, :37].double() @ wo[:, :37].double().T
+        assert rel_rms(ff_total(run_ff(f, h, (a[:, :37].contiguous().cuda(), wo[:, :37].contiguous().cuda()))), odd) < TOL[dtype], (D, M)
 
 
 def test_the_clamp_acts_on_both_sides(dec):
@@ -502,11 +517,11 @@ def test_experts_of_very_unequal_load(dec):
         w["router.b"] = torch.tensor(bias).bfloat16()
         f = ff_module(cfg, w, torch.bfloat16)
         want = o.experts(h.double(), {k: v.double() for k, v in w.items()}, "", cfg)
-        got = ff_total(f(h.cuda()))
+        got = ff_total(run_ff(f, h))
         assert rel_rms(got, want) < TOL[torch.bfloat16]
         out, slots, weight = ops.expert_rows(h.cuda(), f.router, f.router_bias, 2, f.up, f.down, f.gate, plain=True)
         assert rel_rms((out.double()[slots.long()] * weight.double()[..., None]).sum(1), want) < TOL[torch.bfloat16]
-        assert rel_rms(torch.cat([ff_total(f(h[i:i + 7].cuda())) for i in range(0, 70, 7)]), want[:70]) < TOL[torch.bfloat16]
+        assert rel_rms(torch.cat([ff_total(run_ff(f, h[i:i + 7])) for i in range(0, 70, 7)]), want[:70]) < TOL[torch.bfloat16]
 
 
 @pytest.mark.parametrize("rows,G,N,K", [(300, 1, 512, 192), (129, 1, 16, 8), (1000, 3, 272, 200), (70, 5, 48, 1000), (5000, 2, 1040, 64), (64, 1, 256, 64)])
