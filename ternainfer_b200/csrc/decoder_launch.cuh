@@ -6,6 +6,9 @@
 #include <stdio.h>
 
 #include <algorithm>
+#include <map>
+#include <mutex>
+#include <utility>
 
 #include "decoder_ops.h"
 
@@ -31,11 +34,33 @@ inline int bad(int code, const char* what) {
 }
 inline bool misaligned(const void* p, unsigned n) { return (reinterpret_cast<uintptr_t>(p) & (n - 1)) != 0; }
 
+// Attributes of a kernel that depend on its shared memory, set when they change.
+//  * Requests above 48 KB in all (what a kernel has beside it in fixed arrays counts) have to be announced.
+//  * Kernels of a decode step ask for a moderate share of the SM's memory as shared memory.  Without a wish of their own
+//    they would run in whatever split the last kernel with a large request left behind, and with most of the SM's
+//    memory taken away from L1 far fewer weight loads are in flight.
+inline bool set_attributes(const void* kernel, size_t smem, int pdl) {
+    static std::mutex lock;
+    static std::map<std::pair<int, const void*>, std::pair<size_t, int>> done;
+    int dev = 0;
+    cudaGetDevice(&dev);
+    const int share = pdl && smem <= 100 * 1024 ? (int)std::max<size_t>(30, 200 * (smem + 12 * 1024) / (228 * 1024)) : 0;   // two CTAs
+    const std::lock_guard<std::mutex> guard(lock);
+    auto& d = done[{dev, kernel}];
+    if (smem > std::max<size_t>(d.first, 16 * 1024)) {
+        if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) return false;
+        d.first = smem;
+    }
+    if (share > d.second) {
+        if (cudaFuncSetAttribute(kernel, cudaFuncAttributePreferredSharedMemoryCarveout, std::min(share, 100)) != cudaSuccess) return false;
+        d.second = share;
+    }
+    return true;
+}
+
 template <typename... P, typename... Q>
 inline int launch(void (*kernel)(P...), dim3 grid, int threads, size_t smem, int pdl, void* stream, int cluster, Q... args) {
-    if (smem > 16 * 1024 &&   // (what a kernel has beside it in fixed arrays counts towards the 48 KB that need no request)
-        cudaFuncSetAttribute(reinterpret_cast<const void*>(kernel), cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
-        return bad(DECODER_LAUNCH, "shared memory request refused");
+    if (!set_attributes(reinterpret_cast<const void*>(kernel), smem, pdl)) return bad(DECODER_LAUNCH, "shared memory request refused");
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = grid;
     cfg.blockDim = dim3(threads, 1, 1);

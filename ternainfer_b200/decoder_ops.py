@@ -336,9 +336,10 @@ def latent_attention_step(qa, cache, w_uv, sink, pos, T: int, vdim: int, scale: 
     R, slots = w_uv.shape[1], cache.shape[1]
     if splits is None:      # as many ranges of at least 32 keys as the chip holds at a time
         sms = torch.cuda.get_device_properties(qa.device).multi_processor_count
-        ranges = max(1, min(sms // (M * -(-H // 32)), -(-slots // 32)))
-        cluster = min(8 if M * -(-H // 32) * ranges <= 64 else 4, ranges)    # few CTAs: larger clusters still find room
-        splits = (ranges // cluster, cluster)
+        rows, most = M * -(-H // 32), max(1, -(-slots // 32))
+        # clusters of eight leave few parts to join, but only about two thirds of the chip can be filled with them
+        cluster = min(8 if rows <= 2 else 4, most)
+        splits = (max(1, min((sms * 2 // 3 if cluster == 8 else sms) // rows, most) // cluster), cluster)
     parts, cluster = splits
     part = torch.empty((M, H, parts, R), dtype=torch.float32, device=qa.device)
     ml = torch.empty((M, H, parts, 2), dtype=torch.float32, device=qa.device)
