@@ -1,4 +1,4 @@
-"""GPU: the kernels of libdecoderops.so and the Kepovik model on them against the plain CPU restatement.
+"""GPU: the kernels of the Kepovik decoder and the model on them against the plain CPU restatement.
 
 Random weights hide a wrong key among hundreds, so the attention tests give chosen keys and queries one large
 common component: the chosen key's weight is then near one and its value dominates the output, and a key that
